@@ -96,6 +96,7 @@ struct DecodeParams {
     float scale_over_cap;
     const float* distance_bias;  // fp32 [n_heads, bias_rows] (nullptr: none), see PlAttentionExtras
     int bias_rows;
+    const float* distance_slopes;  // fp32 [n_heads] (nullptr: none)
 };
 
 // In-cluster merge: outputs are counted in groups of four dims ("vecs"); rank r owns
@@ -203,6 +204,12 @@ __device__ __forceinline__ void attention_decode_share(const DecodeParams& p, un
         o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.0f;
     }
     float m_lo = -INFINITY, m_hi = -INFINITY, l_lo = 0.0f, l_hi = 0.0f;
+    // The linear bias of this thread's two heads, in the exponent's units per token of distance.
+    float slope_lo = 0.0f, slope_hi = 0.0f;
+    if (EXTRAS && p.distance_slopes != nullptr) {
+        slope_lo = p.distance_slopes[kv_head * p.group + min(g, p.group - 1)] * 1.4426950408889634f;
+        slope_hi = p.distance_slopes[kv_head * p.group + min(g + 8, p.group - 1)] * 1.4426950408889634f;
+    }
 
     // The first tiles are asked for before the wait on earlier kernels: they hold keys of
     // earlier steps, which no kernel of this step writes. Only the tile with the newest
@@ -345,6 +352,9 @@ __device__ __forceinline__ void attention_decode_share(const DecodeParams& p, un
                     const int d = min(ctx - 1 - key, p.bias_rows - 1);
                     scaled = fmaf(__ldg(p.distance_bias + static_cast<int64_t>(kv_head * p.group + hg) * p.bias_rows + d),
                                   1.4426950408889634f, scaled);
+                }
+                if (EXTRAS && p.distance_slopes != nullptr) {
+                    scaled = fmaf(e < 2 ? slope_lo : slope_hi, static_cast<float>(key - (ctx - 1)), scaled);
                 }
                 s[j][e] = ok ? scaled : -INFINITY;
             }
@@ -1047,9 +1057,11 @@ int run_attention_decode(bool allow_cluster, const void* q, int64_t q_row_stride
     p.cap_log2 = p.scale_over_cap = 0.0f;
     p.distance_bias = nullptr;
     p.bias_rows = 0;
+    p.distance_slopes = nullptr;
     if (extras != nullptr) {
         p.distance_bias = extras->distance_bias;
         p.bias_rows = extras->bias_rows;
+        p.distance_slopes = extras->distance_slopes;
         PL_REQUIRE(p.distance_bias == nullptr || p.bias_rows > 0, "attention_decode: a distance bias needs rows");
         PL_REQUIRE(items == nullptr && tile_max == nullptr,
                    "attention_decode: sinks, gates and split weights are not taken over a work list or with attention mass");

@@ -51,6 +51,7 @@ struct PrefillParams {
     float scale_over_cap;
     const float* distance_bias;  // fp32 [n_heads, bias_rows] (nullptr: none), see PlAttentionExtras
     int bias_rows;
+    const float* distance_slopes;  // fp32 [n_heads] (nullptr: none), see PlAttentionExtras
     int n_heads;
 };
 
@@ -182,6 +183,8 @@ __global__ void __launch_bounds__(kThreads, 2) attention_prefill_kernel(const Pr
             }
             float tile_lo = -INFINITY, tile_hi = -INFINITY;
             // (with a bias by distance: the table's entry for this head, in the exponent's units)
+            const float slope_log2 =
+                EXTRAS && p.distance_slopes != nullptr ? p.distance_slopes[head] * 1.4426950408889634f : 0.0f;
             auto exponent_of = [&](float raw, int key, int pos) {
                 if (!EXTRAS) {
                     return raw * p.scale_log2;
@@ -190,6 +193,9 @@ __global__ void __launch_bounds__(kThreads, 2) attention_prefill_kernel(const Pr
                 if (p.distance_bias != nullptr) {
                     const int d = min(max(pos - key, 0), p.bias_rows - 1);
                     x = fmaf(__ldg(p.distance_bias + static_cast<int64_t>(head) * p.bias_rows + d), 1.4426950408889634f, x);
+                }
+                if (p.distance_slopes != nullptr) {
+                    x = fmaf(slope_log2, static_cast<float>(key - pos), x);
                 }
                 return x;
             };
@@ -330,7 +336,7 @@ int launch_prefill_build(const PrefillParams& p, int n_tiles, int n_heads, cudaS
 template <int HD>
 int launch_prefill(const PrefillParams& p, int n_tiles, int n_heads, cudaStream_t stream) {
     const bool extras = p.sinks != nullptr || p.gate != nullptr || p.split_weights || p.v_pool == p.k_pool ||
-                        p.cap_log2 > 0.0f || p.distance_bias != nullptr;
+                        p.cap_log2 > 0.0f || p.distance_bias != nullptr || p.distance_slopes != nullptr;
     return extras ? launch_prefill_build<HD, true>(p, n_tiles, n_heads, stream)
                   : launch_prefill_build<HD, false>(p, n_tiles, n_heads, stream);
 }
@@ -393,6 +399,7 @@ PL_API int pl_attention_prefill(const void* q, int64_t q_row_stride, const void*
     p.split_weights = extras != nullptr ? extras->split_weights : 0;
     p.distance_bias = extras != nullptr ? extras->distance_bias : nullptr;
     p.bias_rows = extras != nullptr ? extras->bias_rows : 0;
+    p.distance_slopes = extras != nullptr ? extras->distance_slopes : nullptr;
     p.n_heads = n_heads;
     PL_REQUIRE(p.distance_bias == nullptr || p.bias_rows > 0, "attention_prefill: a distance bias needs rows");
     p.cap_log2 = p.scale_over_cap = 0.0f;

@@ -78,12 +78,19 @@ struct TcPrefillParams {
     float* mass_part;            // zero before the launch
     int mass_pages;
     float scale;
-    // A bias by distance (the build with BIAS only): fp32 [n_heads, bias_rows], a head's entries side by
+    // A bias by distance (the builds with kBiasTable only): fp32 [n_heads, bias_rows], a head's entries side by
     // side; bias[h, min(d, bias_rows - 1)] joins head h's scaled score of a key d tokens before the query.
     const float* bias;
     int bias_rows;
     float inv_scale;  // the bias enters the raw products: bias / scale, so that (s + bias / scale) * scale is the biased score
+    // A linear bias (the builds with kBiasSlopes only): fp32 [n_heads], slopes[h] * d is taken off head h's scaled
+    // score; and a sink per head, exp(sinks[h]) in the row's denominator (nullptr: none).
+    const float* slopes;
+    const float* sinks;
 };
+
+// What a build adds to its scores by distance.
+enum BiasKind : int { kBiasNone = 0, kBiasTable = 1, kBiasSlopes = 2 };
 
 // What pl_attention_prefill_tcgen05 needs to measure attention mass: the rows' weights,
 // zeroed scratch of n_tiles * n_heads * 8 * pages floats (pages >= the block table's
@@ -145,7 +152,7 @@ __device__ __forceinline__ uint64_t smem_descriptor_mn(const void* tile, uint32_
 // WIDE (with HEADS == 2, for odd groups): the two "heads" of the CTA are the two
 // 128-row halves of one tile of up to 256 rows of ONE head: they share K and V just
 // the same, and everything that says head `hs` below means rows 128 hs ... of it.
-template <int HD, int HEADS, bool WIDE, bool BIAS = false>
+template <int HD, int HEADS, bool WIDE, int BIAS = kBiasNone>
 __global__ void __launch_bounds__(kThreadsTc, 1)
 attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                                  const __grid_constant__ CUtensorMap map_v, const TcPrefillParams p) {
@@ -451,6 +458,9 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
         const int first = p.window > 0 ? pos - p.window + 1 : 0;
         float m = -INFINITY, l = 0.0f;  // m: the base of the exponents in use (lags the true maximum)
         bool ok = true;
+        // (kBiasSlopes: the head's slope in the exponent's units and in those of the raw products)
+        const float slope = BIAS == kBiasSlopes ? p.slopes[head] : 0.0f;
+        const float slope_log2 = slope * 1.4426950408889634f, slope_raw = slope * p.inv_scale;
         const float mass_weight = p.mass_part != nullptr && rr < n_rows ? p.query_weights[row0 + rr] : 0.0f;
         if constexpr (kTurns) {
             // This thread's row of Q into tensor memory, where the first product reads its A
@@ -508,13 +518,28 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
                 mbar_arrive(&s_free[hs][b]);
             }
             const int key0 = (j0 + j) * kKeys + part * kMyKeys;
-            if constexpr (BIAS) {
+            if constexpr (BIAS == kBiasTable) {
                 // this row's bias at every key's distance (neighbouring keys, neighbouring entries of the head's row)
                 const float* bias_row = p.bias + static_cast<int64_t>(head) * p.bias_rows;
 #pragma unroll
                 for (int c = 0; c < kMyKeys; ++c) {
                     const int d = min(max(pos - (key0 + c), 0), p.bias_rows - 1);
                     s[c] = fmaf(__ldg(bias_row + d), p.inv_scale, s[c]);
+                }
+            }
+            // A linear bias is slope * (key - pos) = slope * c + slope * (key0 - pos): the part that differs between the
+            // tile's keys joins the raw products (one packed multiply-add a pair), the rest is one number per row and
+            // tile that joins the maximum and the exponents' base.
+            float tile_shift = 0.0f;
+            if constexpr (BIAS == kBiasSlopes) {
+                tile_shift = slope_log2 * static_cast<float>(key0 - pos);
+                const float2 step = make_float2(slope_raw, slope_raw);
+#pragma unroll
+                for (int c = 0; c < kMyKeys; c += 2) {
+                    const float2 biased = __ffma2_rn(make_float2(static_cast<float>(c), static_cast<float>(c + 1)), step,
+                                                     make_float2(s[c], s[c + 1]));
+                    s[c] = biased.x;
+                    s[c + 1] = biased.y;
                 }
             }
             const bool edge = (j0 + j) * kKeys + kKeys - 1 > pos0 ||
@@ -572,6 +597,9 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
                 }
             }
             float tile_max = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])) * p.scale_log2;
+            if constexpr (BIAS == kBiasSlopes) {
+                tile_max += tile_shift;
+            }
             if (HEADS == 1) {
                 // The row's maximum over both halves: exchange through shared memory.
                 half_max[b][wg * kRows + r] = tile_max;
@@ -608,7 +636,7 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
                 tcgen05_wait_st();
                 tcgen05_fence_before();
             }
-            const float minus_base = m == -INFINITY ? 0.0f : -m;
+            const float minus_base = m == -INFINITY ? 0.0f : BIAS == kBiasSlopes ? tile_shift - m : -m;
             // Exponentials two at a time (packed fp32 arithmetic). Of every four pairs, kCubic
             // take the cubic on the FMA pipe and the rest the special-function unit (one
             // exponential per eight cycles and warp). Measured: at head size 64, where the
@@ -677,7 +705,8 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
                 }
             }
         } else if (ok) {
-            const float inv = l > 0.0f ? 1.0f / l : 0.0f;
+            const float inv = BIAS == kBiasSlopes ? pl_attention_row_factor(m, l, p.sinks, nullptr, 0, 0, head)
+                                                  : (l > 0.0f ? 1.0f / l : 0.0f);
             __nv_bfloat16* dst = p.out + (row0 + rr) * p.out_row_stride + static_cast<int64_t>(head) * HD +
                 part * kMyDims;
 #pragma unroll
@@ -773,7 +802,7 @@ __global__ void __launch_bounds__(256) attention_prefill_merge_kernel(const TcPr
             }
         }
     }
-    const float inv = total > 0.0f ? 1.0f / total : 0.0f;
+    const float inv = pl_attention_row_factor(top, total, p.sinks, nullptr, 0, 0, head);
     __nv_bfloat16* dst = p.out + (tile.x + r) * p.out_row_stride + static_cast<int64_t>(head) * HD + lane * kPer;
 #pragma unroll
     for (int i = 0; i < kPer; i += 2) {
@@ -834,7 +863,7 @@ __global__ void attention_mass_fold_prefill_kernel(const TcPrefillParams p, int 
     }
 }
 
-template <int HD, int HEADS, bool WIDE, bool BIAS = false>
+template <int HD, int HEADS, bool WIDE, int BIAS = kBiasNone>
 int launch_tc_prefill(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const TcPrefillParams& p,
                       int n_tiles, int n_heads, cudaStream_t stream) {
     constexpr int smem = (HEADS == 2 ? 0 : kRows * HD * 2) + stages_kv(HEADS) * 2 * kKeys * HD * 2 + 1024;
@@ -891,8 +920,8 @@ static int run_tc_prefill(const void* q, int64_t q_row_stride, int n_tokens, con
                           int n_pages, const int32_t* table, int table_width, const int32_t* tiles,
                           int n_tiles, void* out, int64_t out_row_stride, int n_heads, int n_kv_heads,
                           int head_dim, int window, float scale, int n_splits, float* scratch,
-                          int wide, const PlPrefillMass* mass, const float* bias, int bias_rows, int32_t* status,
-                          cudaStream_t stream) {
+                          int wide, const PlPrefillMass* mass, const float* bias, int bias_rows, const float* slopes,
+                          const float* sinks, int32_t* status, cudaStream_t stream) {
     PL_REQUIRE(n_tiles >= 0 && n_heads > 0 && n_kv_heads > 0 && n_heads % n_kv_heads == 0 && n_tokens > 0,
                "attention_prefill_tcgen05: bad sizes tiles=%d heads=%d kv_heads=%d tokens=%d", n_tiles, n_heads,
                n_kv_heads, n_tokens);
@@ -957,6 +986,10 @@ static int run_tc_prefill(const void* q, int64_t q_row_stride, int n_tokens, con
     p.bias = bias;
     p.bias_rows = bias_rows;
     p.inv_scale = 1.0f / scale;
+    p.slopes = slopes;
+    p.sinks = sinks;
+    PL_REQUIRE(slopes == nullptr ? sinks == nullptr : bias == nullptr && mass == nullptr,
+               "attention_prefill_tcgen05: a linear bias is taken without a table and without attention mass, a sink only with it");
     if (bias != nullptr) {
         PL_REQUIRE(pairs && mass == nullptr && bias_rows > 0,
                    "attention_prefill_tcgen05: a bias by distance is taken with two heads of a kv head per CTA (an even "
@@ -984,8 +1017,15 @@ static int run_tc_prefill(const void* q, int64_t q_row_stride, int n_tokens, con
     }
     int code;
     if (bias != nullptr) {
-        code = head_dim == 64 ? launch_tc_prefill<64, 2, false, true>(mq, mk, mv, p, n_tiles, n_heads, stream)
-                              : launch_tc_prefill<128, 2, false, true>(mq, mk, mv, p, n_tiles, n_heads, stream);
+        code = head_dim == 64 ? launch_tc_prefill<64, 2, false, kBiasTable>(mq, mk, mv, p, n_tiles, n_heads, stream)
+                              : launch_tc_prefill<128, 2, false, kBiasTable>(mq, mk, mv, p, n_tiles, n_heads, stream);
+    } else if (slopes != nullptr && head_dim == 64) {
+        // (odd groups: always two halves of a tile per CTA, whatever the tiles' rows)
+        code = pairs ? launch_tc_prefill<64, 2, false, kBiasSlopes>(mq, mk, mv, p, n_tiles, n_heads, stream)
+                     : launch_tc_prefill<64, 2, true, kBiasSlopes>(mq, mk, mv, p, n_tiles, n_heads, stream);
+    } else if (slopes != nullptr) {
+        code = pairs ? launch_tc_prefill<128, 2, false, kBiasSlopes>(mq, mk, mv, p, n_tiles, n_heads, stream)
+                     : launch_tc_prefill<128, 2, true, kBiasSlopes>(mq, mk, mv, p, n_tiles, n_heads, stream);
     } else if (head_dim == 64) {
         code = pairs ? launch_tc_prefill<64, 2, false>(mq, mk, mv, p, n_tiles, n_heads, stream)
             : wide   ? launch_tc_prefill<64, 2, true>(mq, mk, mv, p, n_tiles, n_heads, stream)
@@ -1015,7 +1055,7 @@ PL_API int pl_attention_prefill_tcgen05(const void* q, int64_t q_row_stride, int
                                         int wide, const PlPrefillMass* mass, int32_t* status, cudaStream_t stream) {
     return run_tc_prefill(q, q_row_stride, n_tokens, k_pool, v_pool, page_stride, head_stride, page_size, n_pages, table,
                           table_width, tiles, n_tiles, out, out_row_stride, n_heads, n_kv_heads, head_dim, window, scale,
-                          n_splits, scratch, wide, mass, nullptr, 0, status, stream);
+                          n_splits, scratch, wide, mass, nullptr, 0, nullptr, nullptr, status, stream);
 }
 
 // The same with a bias by distance: bias fp32 [n_heads, bias_rows] (a head's entries side by side);
@@ -1031,5 +1071,21 @@ PL_API int pl_attention_prefill_tcgen05_bias(const void* q, int64_t q_row_stride
     PL_REQUIRE(bias != nullptr && bias_rows > 0, "attention_prefill_tcgen05_bias: needs a bias table");
     return run_tc_prefill(q, q_row_stride, n_tokens, k_pool, v_pool, page_stride, head_stride, page_size, n_pages, table,
                           table_width, tiles, n_tiles, out, out_row_stride, n_heads, n_kv_heads, head_dim, window, scale,
-                          n_splits, scratch, 0, nullptr, bias, bias_rows, status, stream);
+                          n_splits, scratch, 0, nullptr, bias, bias_rows, nullptr, nullptr, status, stream);
+}
+
+// The same with a linear bias and, optionally, a sink: slopes fp32 [n_heads], slopes[h] * d is taken off head h's
+// scaled score of a key d tokens before the query; sinks fp32 [n_heads] (may be nullptr), exp(sinks[h]) joins head
+// h's denominator. Any GQA group (an odd one takes tiles of up to 256 rows); no attention mass.
+PL_API int pl_attention_prefill_tcgen05_slopes(const void* q, int64_t q_row_stride, int n_tokens, const void* k_pool,
+                                               const void* v_pool, int64_t page_stride, int64_t head_stride,
+                                               int page_size, int n_pages, const int32_t* table, int table_width,
+                                               const int32_t* tiles, int n_tiles, void* out, int64_t out_row_stride,
+                                               int n_heads, int n_kv_heads, int head_dim, int window, float scale,
+                                               int n_splits, float* scratch, const float* slopes, const float* sinks,
+                                               int32_t* status, cudaStream_t stream) {
+    PL_REQUIRE(slopes != nullptr, "attention_prefill_tcgen05_slopes: needs the heads' slopes");
+    return run_tc_prefill(q, q_row_stride, n_tokens, k_pool, v_pool, page_stride, head_stride, page_size, n_pages, table,
+                          table_width, tiles, n_tiles, out, out_row_stride, n_heads, n_kv_heads, head_dim, window, scale,
+                          n_splits, scratch, n_heads / n_kv_heads % 2, nullptr, nullptr, 0, slopes, sinks, status, stream);
 }

@@ -160,7 +160,9 @@ __device__ __forceinline__ float pl_block_max(float v, float* scratch) {
 // lost), so the weights keep 16 mantissa bits instead of 8. softcap > 0: every scaled score s
 // becomes softcap * tanh(s / softcap) before the softmax. distance_bias: fp32 [n_heads, bias_rows]
 // (a head's entries side by side); distance_bias[h, min(d, bias_rows - 1)] joins head h's scaled (and
-// capped) score of a key d tokens before the query; the scale does not touch it.
+// capped) score of a key d tokens before the query; the scale does not touch it. distance_slopes: fp32
+// [n_heads]; distance_slopes[h] * d is taken off head h's scaled (and capped) score of a key d tokens
+// before the query, for any d (a linear bias without a table's end).
 struct PlAttentionExtras {
     const float* sinks;
     const void* gate;
@@ -169,6 +171,7 @@ struct PlAttentionExtras {
     float softcap;
     const float* distance_bias;
     int bias_rows;
+    const float* distance_slopes;
 };
 
 // A raw score on its way into the base-2 softmax: times scale * log2 e, or with a cap

@@ -479,3 +479,39 @@ PL_API int pl_bias_act(const void* in, int64_t in_row_stride, const void* bias, 
     PL_CHECK_LAUNCH("bias_act");
     return 0;
 }
+
+namespace {
+
+// x = cap * tanh(x * scale / cap), in place (four elements a thread, the rest one by one).
+__global__ void capped_scale_kernel(float* __restrict__ x, int64_t n, float scale_over_cap, float cap) {
+    pl_grid_trigger();
+    pl_grid_wait();
+    const int64_t quads = n / 4;
+    const int64_t first = blockIdx.x * static_cast<int64_t>(blockDim.x) + threadIdx.x;
+    const int64_t step = static_cast<int64_t>(gridDim.x) * blockDim.x;
+    for (int64_t i = first; i < quads; i += step) {
+        const float4 v = pl_load4(x + 4 * i);
+        pl_store4(x + 4 * i, make_float4(cap * tanhf(v.x * scale_over_cap), cap * tanhf(v.y * scale_over_cap),
+                                         cap * tanhf(v.z * scale_over_cap), cap * tanhf(v.w * scale_over_cap)));
+    }
+    for (int64_t i = 4 * quads + first; i < n; i += step) {
+        x[i] = cap * tanhf(x[i] * scale_over_cap);
+    }
+}
+
+}  // namespace
+
+// x fp32 [n], 16-byte aligned: x = cap * tanh(x * scale / cap) in place (an output head's logit scale and cap).
+PL_API int pl_capped_scale(float* x, int64_t n, float scale, float cap, cudaStream_t stream) {
+    PL_REQUIRE(n >= 0 && cap > 0.0f, "capped_scale: bad arguments n=%lld cap=%g", static_cast<long long>(n),
+               static_cast<double>(cap));
+    PL_REQUIRE((reinterpret_cast<uintptr_t>(x) & 15) == 0, "capped_scale: the logits must start on 16 bytes");
+    if (n == 0) {
+        return 0;
+    }
+    const int threads = 256;
+    const int blocks = static_cast<int>(std::min<int64_t>((n / 4 + threads) / threads, 148 * 8));
+    pl_launch_overlapped(capped_scale_kernel, dim3(blocks), dim3(threads), 0, stream, x, n, scale / cap, cap);
+    PL_CHECK_LAUNCH("capped_scale");
+    return 0;
+}

@@ -2,6 +2,8 @@
 // activation, and an output gate per element.
 //
 //   gated_act:     out[t, i] = act(in[t, i]) * in[t, width + i]      act: silu or the tanh form of GELU
+//                  or the clamped unit: g = min(w in[t, i], limit), u = clamp(w in[t, width + i], -limit, limit),
+//                  out = g sigmoid(1.702 g) (u + 1), where w is a weight of the row (1 without one)
 //   sigmoid_gate:  x[t, i]  *= sigmoid(gate[t, i])
 //   sigmoid_gate_heads:  x[t, h, :] *= sigmoid(gate[t, h])     one gate per head
 //
@@ -10,7 +12,18 @@
 
 #include <algorithm>
 
+#include "gate_units.cuh"
+
 namespace {
+
+// What a row's gate and up values become. The row's weight (only the clamped unit takes one) multiplies both: the
+// weight of a routed expert's input, which a linear map carries through.
+struct GateParams {
+    int act;      // 0: silu, 1: the tanh form of GELU, 2: the clamped unit
+    float limit;  // (clamped unit)
+    const float* row_weights;  // fp32 or nullptr
+    const int32_t* row_index;  // row t takes row_weights[row_index[t]] (nullptr: row_weights[t])
+};
 
 __device__ __forceinline__ float gate_activation(float z, int act) {
     if (act == 1) {
@@ -21,9 +34,16 @@ __device__ __forceinline__ float gate_activation(float z, int act) {
     return z / (1.0f + expf(-z));
 }
 
+__device__ __forceinline__ float gate_unit(float g, float u, float w, const GateParams& p) {
+    return p.act == 2 ? pl_clamped_unit(w * g, w * u, p.limit) : gate_activation(g, p.act) * u;
+}
+__device__ __forceinline__ float row_weight(const GateParams& p, int64_t t) {
+    return p.row_weights == nullptr ? 1.0f : p.row_weights[p.row_index != nullptr ? p.row_index[t] : t];
+}
+
 template <typename scalar_t>
 __global__ void gated_act_kernel(const scalar_t* __restrict__ in, scalar_t* __restrict__ out, int64_t tokens,
-                                 int width, int act) {
+                                 int width, const GateParams p) {
     pl_grid_trigger();
     pl_grid_wait();
     const int quads = width / 4;  // (the launcher takes this kernel for widths that are multiples of 4)
@@ -34,14 +54,15 @@ __global__ void gated_act_kernel(const scalar_t* __restrict__ in, scalar_t* __re
         const int i = 4 * static_cast<int>(idx - t * quads);
         const float4 g = pl_load4(in + t * 2 * width + i);
         const float4 u = pl_load4(in + t * 2 * width + width + i);
-        pl_store4(out + t * width + i, make_float4(gate_activation(g.x, act) * u.x, gate_activation(g.y, act) * u.y,
-                                                   gate_activation(g.z, act) * u.z, gate_activation(g.w, act) * u.w));
+        const float w = row_weight(p, t);
+        pl_store4(out + t * width + i, make_float4(gate_unit(g.x, u.x, w, p), gate_unit(g.y, u.y, w, p),
+                                                   gate_unit(g.z, u.z, w, p), gate_unit(g.w, u.w, w, p)));
     }
 }
 
 template <typename scalar_t>
 __global__ void gated_act_scalar_kernel(const scalar_t* __restrict__ in, scalar_t* __restrict__ out, int64_t tokens,
-                                        int width, int act) {
+                                        int width, const GateParams p) {
     pl_grid_trigger();
     pl_grid_wait();
     const int64_t total = tokens * width;
@@ -49,7 +70,8 @@ __global__ void gated_act_scalar_kernel(const scalar_t* __restrict__ in, scalar_
          idx += static_cast<int64_t>(gridDim.x) * blockDim.x) {
         const int64_t t = idx / width;
         const int i = static_cast<int>(idx - t * width);
-        pl_store(out + idx, gate_activation(pl_load(in + t * 2 * width + i), act) * pl_load(in + t * 2 * width + width + i));
+        pl_store(out + idx, gate_unit(pl_load(in + t * 2 * width + i), pl_load(in + t * 2 * width + width + i),
+                                      row_weight(p, t), p));
     }
 }
 
@@ -114,10 +136,14 @@ __global__ void sigmoid_gate_heads_kernel(scalar_t* __restrict__ x, int64_t x_st
 }  // namespace
 
 // in [T, 2 * width] (gate columns, then up columns), out [T, width], both dense, in the
-// engine's dtype. act 0: silu, 1: the tanh form of GELU.
-PL_API int pl_gated_act(const void* in, void* out, int n_tokens, int width, int act, int dtype, cudaStream_t stream) {
-    PL_REQUIRE(n_tokens >= 0 && width > 0 && (act == 0 || act == 1), "gated_act: bad arguments tokens=%d width=%d "
+// engine's dtype. act 0: silu, 1: the tanh form of GELU, 2: the clamped unit with `limit` and, optionally, a weight a
+// row (row_weights fp32; row_index int32 [T] or nullptr).
+PL_API int pl_gated_act(const void* in, void* out, int n_tokens, int width, int act, float limit, const float* row_weights,
+                        const int32_t* row_index, int dtype, cudaStream_t stream) {
+    PL_REQUIRE(n_tokens >= 0 && width > 0 && act >= 0 && act <= 2, "gated_act: bad arguments tokens=%d width=%d "
                "act=%d", n_tokens, width, act);
+    PL_REQUIRE(act == 2 || row_weights == nullptr, "gated_act: only the clamped unit takes a weight a row");
+    const GateParams p = {act, limit, row_weights, row_index};
     if (n_tokens == 0) {
         return 0;
     }
@@ -129,10 +155,10 @@ PL_API int pl_gated_act(const void* in, void* out, int n_tokens, int width, int 
     PL_DISPATCH_DTYPE(dtype, "gated_act", {
         if (quads) {
             pl_launch_overlapped(gated_act_kernel<scalar_t>, dim3(blocks), dim3(threads), 0, stream,
-                                 static_cast<const scalar_t*>(in), static_cast<scalar_t*>(out), n_tokens, width, act);
+                                 static_cast<const scalar_t*>(in), static_cast<scalar_t*>(out), n_tokens, width, p);
         } else {
             pl_launch_overlapped(gated_act_scalar_kernel<scalar_t>, dim3(blocks), dim3(threads), 0, stream,
-                                 static_cast<const scalar_t*>(in), static_cast<scalar_t*>(out), n_tokens, width, act);
+                                 static_cast<const scalar_t*>(in), static_cast<scalar_t*>(out), n_tokens, width, p);
         }
     });
     PL_CHECK_LAUNCH("gated_act");

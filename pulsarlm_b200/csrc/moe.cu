@@ -7,11 +7,14 @@
 // `group_top` largest choice scores (1: its largest), and only experts of the `keep` best
 // groups can be chosen (the others count as minus infinity). The `top` largest choice scores
 // are chosen (ties go to the lower index); their weights are their scores s (without the
-// correction), with `renormalise` over the chosen scores' sum (+ 1e-20). One block per token.
+// correction), with `renormalise` over the chosen scores' sum (+ 1e-20). One block per token. With
+// `shared_gate` the router has one row more: sigmoid of its logit is the token's weight for a shared expert.
 //
 // Experts (pl_moe_gate_up, pl_moe_down): expert e of a token computes W_down,e (silu(W_gate,e h)
 // * (W_up,e h)); pl_moe_up takes the place of pl_moe_gate_up for experts without a gate, W_down,e
-// act(W_up,e h) with act the square of relu. The first kernel takes a (token, chosen expert) pair per block row and writes
+// act(W_up,e h) with act the square of relu. With `clamped` the unit is gate_units.cuh's, and a pair's weight, where
+// given, multiplies the expert's input (its gate and up products: a linear map carries the weight through) instead of
+// its output. The first kernel takes a (token, chosen expert) pair per block row and writes
 // the gated activation, a warp per feature (both rows of the feature read with 16-byte loads,
 // the lanes' shares added in a fixed order); the second takes a token per block row and adds
 // up its experts' down projections times their weights, plus an optional row that every
@@ -24,6 +27,7 @@
 // steps: counts per expert, their running sums, and for every pair its row in that order.
 // One block.
 #include "common.cuh"
+#include "gate_units.cuh"
 
 namespace {
 
@@ -75,13 +79,15 @@ template <typename scalar_t, int TOKENS>
 __global__ void __launch_bounds__(512, TOKENS > 1 ? 2 : 1) moe_route_kernel(const scalar_t* __restrict__ h, int64_t h_stride, const float* __restrict__ router,
                                  const float* __restrict__ correction, int32_t* __restrict__ ids,
                                  float* __restrict__ weights, int n_tokens, int hidden, int n_experts, int top,
-                                 int n_groups, int keep, int sigmoid_scores, int group_top, int renormalise) {
+                                 int n_groups, int keep, int sigmoid_scores, int group_top, int renormalise,
+                                 float* __restrict__ shared_weights) {
     pl_grid_trigger();
     pl_grid_wait();
     extern __shared__ float shared[];
     float* rows = shared;                                   // [TOKENS][hidden]
-    float* scores = rows + TOKENS * hidden;                 // [TOKENS][n_experts]  s
-    float* choices = scores + TOKENS * n_experts;           // [TOKENS][n_experts]  s + correction, -inf once taken or shut out
+    const int n_rows = n_experts + (shared_weights != nullptr ? 1 : 0);  // (a shared expert's gate is the last row)
+    float* scores = rows + TOKENS * hidden;                 // [TOKENS][n_rows]  s
+    float* choices = scores + TOKENS * n_rows;              // [TOKENS][n_experts]  s + correction, -inf once taken or shut out
     float* group_scores = choices + TOKENS * n_experts;     // [TOKENS][n_groups]
     const int t0 = blockIdx.x * TOKENS;
     const int here = min(TOKENS, n_tokens - t0);
@@ -115,7 +121,7 @@ __global__ void __launch_bounds__(512, TOKENS > 1 ? 2 : 1) moe_route_kernel(cons
     }
     __syncthreads();
     const bool vectors = (hidden & 3) == 0 && (reinterpret_cast<uintptr_t>(router) & 15) == 0;
-    for (int e = warp; e < n_experts; e += warps) {
+    for (int e = warp; e < n_rows; e += warps) {
         const float* w = router + static_cast<int64_t>(e) * hidden;
         float z[TOKENS];
 #pragma unroll
@@ -160,7 +166,7 @@ __global__ void __launch_bounds__(512, TOKENS > 1 ? 2 : 1) moe_route_kernel(cons
         for (int r = 0; r < TOKENS; ++r) {
             const float total = pl_warp_sum(z[r]);
             if (lane == 0) {
-                scores[r * n_experts + e] = total;
+                scores[r * n_rows + e] = total;
             }
         }
     }
@@ -169,9 +175,12 @@ __global__ void __launch_bounds__(512, TOKENS > 1 ? 2 : 1) moe_route_kernel(cons
         return;
     }
     const int t = t0 + warp;
-    float* score = scores + warp * n_experts;
+    float* score = scores + warp * n_rows;
     float* choice = choices + warp * n_experts;
     float* group_score = group_scores + warp * n_groups;
+    if (shared_weights != nullptr && lane == 0) {
+        shared_weights[t] = 1.0f / (1.0f + expf(-score[n_experts]));
+    }
     if (sigmoid_scores) {
         for (int e = lane; e < n_experts; e += 32) {
             const float s = 1.0f / (1.0f + expf(-score[e]));
@@ -386,12 +395,13 @@ __device__ __forceinline__ void warp_dots_two(const scalar_t* __restrict__ w0, c
 
 constexpr int kFeaturesPerWarp = 4;
 
-// Block (pair, feature block): act[pair, f] = silu(gate_e[f] . h) * (up_e[f] . h).
-template <typename scalar_t>
+// Block (pair, feature block): act[pair, f] = silu(gate_e[f] . h) * (up_e[f] . h), or (CLAMPED) the clamped unit of
+// w (gate_e[f] . h) and w (up_e[f] . h), w the pair's weight.
+template <typename scalar_t, bool CLAMPED>
 __global__ void moe_gate_up_kernel(const scalar_t* __restrict__ h, int64_t h_stride,
                                    const scalar_t* __restrict__ gate_up, const int32_t* __restrict__ ids,
                                    scalar_t* __restrict__ act, int hidden, int ff, int top, int n_experts,
-                                   int vectors) {
+                                   int vectors, const float* __restrict__ in_weights, float limit) {
     pl_grid_trigger();
     pl_grid_wait();
     extern __shared__ float row[];  // [hidden]
@@ -399,6 +409,10 @@ __global__ void moe_gate_up_kernel(const scalar_t* __restrict__ h, int64_t h_str
     const int t = pair / top;
     const int e = ids[pair];
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
+    const float in_weight = CLAMPED && in_weights != nullptr ? in_weights[pair] : 1.0f;
+    auto unit = [&](float g, float u) {
+        return CLAMPED ? pl_clamped_unit(in_weight * g, in_weight * u, limit) : silu_f32(g) * u;
+    };
     for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
         row[i] = pl_load(h + t * h_stride + i);
     }
@@ -421,7 +435,7 @@ __global__ void moe_gate_up_kernel(const scalar_t* __restrict__ h, int64_t h_str
                 gl = lane == r ? g[r] : gl;
                 ul = lane == r ? u[r] : ul;
             }
-            pl_store(act + static_cast<int64_t>(pair) * ff + f0 + lane, silu_f32(gl) * ul);
+            pl_store(act + static_cast<int64_t>(pair) * ff + f0 + lane, unit(gl, ul));
         }
         return;
     }
@@ -429,7 +443,7 @@ __global__ void moe_gate_up_kernel(const scalar_t* __restrict__ h, int64_t h_str
         const float g = warp_dot<scalar_t>(weights + static_cast<int64_t>(f) * hidden, row, hidden, vectors, lane);
         const float u = warp_dot<scalar_t>(weights + static_cast<int64_t>(ff + f) * hidden, row, hidden, vectors, lane);
         if (lane == 0) {
-            pl_store(act + static_cast<int64_t>(pair) * ff + f, silu_f32(g) * u);
+            pl_store(act + static_cast<int64_t>(pair) * ff + f, unit(g, u));
         }
     }
 }
@@ -481,12 +495,13 @@ __global__ void moe_up_kernel(const scalar_t* __restrict__ h, int64_t h_stride, 
 
 constexpr int kChannelsPerWarp = 4;
 
-// Block (token, channel block): out[t, c] = sum_j weight[t, j] * (down_{e_j}[c] . act[t, j]) + also[t, c].
+// Block (token, channel block): out[t, c] = sum_j weight[t, j] * (down_{e_j}[c] . act[t, j]) + also_weight[t] * also[t, c]
+// (weights nullptr: all 1; also_weights nullptr: 1).
 template <typename scalar_t>
 __global__ void moe_down_kernel(const scalar_t* __restrict__ act, const scalar_t* __restrict__ down,
                                 const int32_t* __restrict__ ids, const float* __restrict__ weights,
-                                const scalar_t* __restrict__ also, scalar_t* __restrict__ out, int hidden, int ff,
-                                int top, int n_experts, int vectors) {
+                                const scalar_t* __restrict__ also, const float* __restrict__ also_weights,
+                                scalar_t* __restrict__ out, int hidden, int ff, int top, int n_experts, int vectors) {
     pl_grid_trigger();
     pl_grid_wait();
     extern __shared__ float rows[];  // [top][ff]
@@ -525,14 +540,14 @@ __global__ void moe_down_kernel(const scalar_t* __restrict__ act, const scalar_t
                 }
             }
             if (ok0) {
-                const float weight = weights[static_cast<int64_t>(t) * top + j];
+                const float weight = weights != nullptr ? weights[static_cast<int64_t>(t) * top + j] : 1.0f;
 #pragma unroll
                 for (int r = 0; r < kChannelsPerWarp; ++r) {
                     sums[r] = fmaf(weight, dots0[r], sums[r]);
                 }
             }
             if (ok1) {
-                const float weight = weights[static_cast<int64_t>(t) * top + j + 1];
+                const float weight = weights != nullptr ? weights[static_cast<int64_t>(t) * top + j + 1] : 1.0f;
 #pragma unroll
                 for (int r = 0; r < kChannelsPerWarp; ++r) {
                     sums[r] = fmaf(weight, dots1[r], sums[r]);
@@ -547,7 +562,8 @@ __global__ void moe_down_kernel(const scalar_t* __restrict__ act, const scalar_t
             }
             const int c = c0 + lane;
             if (also != nullptr) {
-                sum += pl_load(also + static_cast<int64_t>(t) * hidden + c);
+                const float more = pl_load(also + static_cast<int64_t>(t) * hidden + c);
+                sum = also_weights != nullptr ? fmaf(also_weights[t], more, sum) : sum + more;
             }
             pl_store(out + static_cast<int64_t>(t) * hidden + c, sum);
         }
@@ -561,12 +577,13 @@ __global__ void moe_down_kernel(const scalar_t* __restrict__ act, const scalar_t
                 continue;
             }
             const scalar_t* w = down + (static_cast<int64_t>(e) * hidden + c) * ff;
-            sum = fmaf(weights[static_cast<int64_t>(t) * top + j], warp_dot<scalar_t>(w, rows + j * ff, ff, vectors, lane),
-                       sum);
+            sum = fmaf(weights != nullptr ? weights[static_cast<int64_t>(t) * top + j] : 1.0f,
+                       warp_dot<scalar_t>(w, rows + j * ff, ff, vectors, lane), sum);
         }
         if (lane == 0) {
             if (also != nullptr) {
-                sum += pl_load(also + static_cast<int64_t>(t) * hidden + c);
+                const float more = pl_load(also + static_cast<int64_t>(t) * hidden + c);
+                sum = also_weights != nullptr ? fmaf(also_weights[t], more, sum) : sum + more;
             }
             pl_store(out + static_cast<int64_t>(t) * hidden + c, sum);
         }
@@ -635,20 +652,23 @@ __global__ void moe_gather_kernel(const scalar_t* __restrict__ x, int64_t x_stri
     }
 }
 
-// out[t] = sum_j weight[t, j] * y[row_of_pair[t, j]] + also[t], fp32 sums, one rounding.
+// out[t] = sum_j weight[t, j] * y[row_of_pair[t, j]] + also_weight[t] * also[t], fp32 sums, one rounding (weights and
+// also_weights as in moe_down).
 template <typename scalar_t>
 __global__ void moe_combine_kernel(const scalar_t* __restrict__ y, const int32_t* __restrict__ row_of_pair,
                                    const float* __restrict__ weights, const scalar_t* __restrict__ also,
-                                   scalar_t* __restrict__ out, int hidden, int top, int vectors) {
+                                   const float* __restrict__ also_weights, scalar_t* __restrict__ out, int hidden, int top,
+                                   int vectors) {
     pl_grid_trigger();
     pl_grid_wait();
     const int64_t t = blockIdx.x;
+    const float also_weight = also_weights != nullptr ? also_weights[t] : 1.0f;
     if (vectors) {
         // (the same sums, four channels at a time)
         for (int i = 4 * threadIdx.x; i < hidden; i += 4 * blockDim.x) {
             float4 sum = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
             for (int j = 0; j < top; ++j) {
-                const float weight = weights[t * top + j];
+                const float weight = weights != nullptr ? weights[t * top + j] : 1.0f;
                 const float4 v = pl_load4(y + static_cast<int64_t>(row_of_pair[t * top + j]) * hidden + i);
                 sum.x = fmaf(weight, v.x, sum.x);
                 sum.y = fmaf(weight, v.y, sum.y);
@@ -657,10 +677,10 @@ __global__ void moe_combine_kernel(const scalar_t* __restrict__ y, const int32_t
             }
             if (also != nullptr) {
                 const float4 v = pl_load4(also + t * hidden + i);
-                sum.x += v.x;
-                sum.y += v.y;
-                sum.z += v.z;
-                sum.w += v.w;
+                sum.x = fmaf(also_weight, v.x, sum.x);
+                sum.y = fmaf(also_weight, v.y, sum.y);
+                sum.z = fmaf(also_weight, v.z, sum.z);
+                sum.w = fmaf(also_weight, v.w, sum.w);
             }
             pl_store4(out + t * hidden + i, sum);
         }
@@ -669,10 +689,11 @@ __global__ void moe_combine_kernel(const scalar_t* __restrict__ y, const int32_t
     for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
         float sum = 0.0f;
         for (int j = 0; j < top; ++j) {
-            sum = fmaf(weights[t * top + j], pl_load(y + static_cast<int64_t>(row_of_pair[t * top + j]) * hidden + i), sum);
+            sum = fmaf(weights != nullptr ? weights[t * top + j] : 1.0f,
+                       pl_load(y + static_cast<int64_t>(row_of_pair[t * top + j]) * hidden + i), sum);
         }
         if (also != nullptr) {
-            sum += pl_load(also + t * hidden + i);
+            sum = fmaf(also_weight, pl_load(also + t * hidden + i), sum);
         }
         pl_store(out + t * hidden + i, sum);
     }
@@ -683,10 +704,12 @@ __global__ void moe_combine_kernel(const scalar_t* __restrict__ y, const int32_t
 // h [T, hidden] (h_stride elements between rows) in the engine's dtype; router fp32 [n_experts,
 // hidden]; correction fp32 [n_experts] or null; ids int32 [T, top]; weights fp32 [T, top].
 // sigmoid_scores: s = sigmoid(z) instead of softmax(z); group_top: how many of a group's largest choice
-// scores add up to its score; renormalise: whether the chosen scores are divided by their sum.
+// scores add up to its score; renormalise: whether the chosen scores are divided by their sum. shared_weights (fp32
+// [T], may be nullptr): sigmoid of the logit of one more row of the router, a shared expert's gate.
 PL_API int pl_moe_route(const void* h, int64_t h_stride, const float* router, const float* correction, int32_t* ids,
                         float* weights, int n_tokens, int hidden, int n_experts, int top, int n_groups, int keep,
-                        int sigmoid_scores, int group_top, int renormalise, int dtype, cudaStream_t stream) {
+                        int sigmoid_scores, int group_top, int renormalise, float* shared_weights, int dtype,
+                        cudaStream_t stream) {
     PL_REQUIRE(group_top > 0 && group_top <= kMaxGroupTop, "moe_route: a group's score adds up 1 to %d scores, not %d",
                kMaxGroupTop, group_top);
     PL_REQUIRE(n_tokens >= 0 && hidden > 0 && n_experts > 0 && top > 0 && n_groups > 0 && keep > 0,
@@ -696,7 +719,8 @@ PL_API int pl_moe_route(const void* h, int64_t h_stride, const float* router, co
                n_experts, n_groups, keep);
     PL_REQUIRE(top <= keep * (n_experts / n_groups), "moe_route: %d experts cannot be chosen from %d groups of %d", top,
                keep, n_experts / n_groups);
-    const size_t per_token = (static_cast<size_t>(hidden) + 2 * n_experts + n_groups) * sizeof(float);
+    const size_t per_token =
+        (static_cast<size_t>(hidden) + 2 * n_experts + (shared_weights != nullptr ? 1 : 0) + n_groups) * sizeof(float);
     PL_REQUIRE(per_token <= 200 * 1024, "moe_route: hidden %d and %d experts need too much shared memory", hidden,
                n_experts);
     if (n_tokens == 0) {
@@ -717,7 +741,8 @@ PL_API int pl_moe_route(const void* h, int64_t h_stride, const float* router, co
             cudaFuncSetAttribute(moe_route_kernel<scalar_t, 8>, cudaFuncAttributePreferredSharedMemoryCarveout, 100);
             pl_launch_overlapped(moe_route_kernel<scalar_t, 8>, dim3((n_tokens + 7) / 8), dim3(threads), smem, stream,
                                  static_cast<const scalar_t*>(h), h_stride, router, correction, ids, weights, n_tokens,
-                                 hidden, n_experts, top, n_groups, keep, sigmoid_scores, group_top, renormalise);
+                                 hidden, n_experts, top, n_groups, keep, sigmoid_scores, group_top, renormalise,
+                                 shared_weights);
         } else {
             if (smem > 48 * 1024) {
                 cudaFuncSetAttribute(moe_route_kernel<scalar_t, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize,
@@ -725,16 +750,20 @@ PL_API int pl_moe_route(const void* h, int64_t h_stride, const float* router, co
             }
             pl_launch_overlapped(moe_route_kernel<scalar_t, 1>, dim3(n_tokens), dim3(threads), smem, stream,
                                  static_cast<const scalar_t*>(h), h_stride, router, correction, ids, weights, n_tokens,
-                                 hidden, n_experts, top, n_groups, keep, sigmoid_scores, group_top, renormalise);
+                                 hidden, n_experts, top, n_groups, keep, sigmoid_scores, group_top, renormalise,
+                                 shared_weights);
         }
     });
     PL_CHECK_LAUNCH("moe_route");
     return 0;
 }
 
-// gate_up [n_experts, 2 * ff, hidden] (an expert's gate rows, then its up rows); act [T * top, ff].
+// gate_up [n_experts, 2 * ff, hidden] (an expert's gate rows, then its up rows); act [T * top, ff]. clamped != 0: the
+// clamped unit with `limit`, and in_weights (fp32 [T * top], may be nullptr) on the pairs' gate and up products.
 PL_API int pl_moe_gate_up(const void* h, int64_t h_stride, const void* gate_up, const int32_t* ids, void* act,
-                          int n_tokens, int hidden, int ff, int top, int n_experts, int dtype, cudaStream_t stream) {
+                          int n_tokens, int hidden, int ff, int top, int n_experts, int clamped, float limit,
+                          const float* in_weights, int dtype, cudaStream_t stream) {
+    PL_REQUIRE(clamped || in_weights == nullptr, "moe_gate_up: only the clamped unit takes weights on its input");
     PL_REQUIRE(n_tokens >= 0 && hidden > 0 && ff > 0 && top > 0 && n_experts > 0, "moe_gate_up: bad sizes");
     const size_t smem = static_cast<size_t>(hidden) * sizeof(float);
     PL_REQUIRE(smem <= 200 * 1024, "moe_gate_up: hidden %d is too wide", hidden);
@@ -747,12 +776,13 @@ PL_API int pl_moe_gate_up(const void* h, int64_t h_stride, const void* gate_up, 
     PL_DISPATCH_DTYPE(dtype, "moe_gate_up", {
         const int vectors = hidden % Vec<scalar_t>::kCount == 0 && (reinterpret_cast<uintptr_t>(gate_up) & 15) == 0;
         if (smem > 48 * 1024) {
-            cudaFuncSetAttribute(moe_gate_up_kernel<scalar_t>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                 static_cast<int>(smem));
+            cudaFuncSetAttribute(clamped ? moe_gate_up_kernel<scalar_t, true> : moe_gate_up_kernel<scalar_t, false>,
+                                 cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
         }
-        pl_launch_overlapped(moe_gate_up_kernel<scalar_t>, grid, dim3(warps * 32), smem, stream,
-                             static_cast<const scalar_t*>(h), h_stride, static_cast<const scalar_t*>(gate_up), ids,
-                             static_cast<scalar_t*>(act), hidden, ff, top, n_experts, vectors);
+        pl_launch_overlapped(clamped ? moe_gate_up_kernel<scalar_t, true> : moe_gate_up_kernel<scalar_t, false>, grid,
+                             dim3(warps * 32), smem, stream, static_cast<const scalar_t*>(h), h_stride,
+                             static_cast<const scalar_t*>(gate_up), ids, static_cast<scalar_t*>(act), hidden, ff, top,
+                             n_experts, vectors, in_weights, limit);
     });
     PL_CHECK_LAUNCH("moe_gate_up");
     return 0;
@@ -784,9 +814,10 @@ PL_API int pl_moe_up(const void* h, int64_t h_stride, const void* up, const int3
     return 0;
 }
 
-// act [T * top, ff]; down [n_experts, hidden, ff]; also [T, hidden] or null; out [T, hidden].
+// act [T * top, ff]; down [n_experts, hidden, ff]; weights fp32 [T, top] or null (all 1); also [T, hidden] or null, times
+// also_weights (fp32 [T] or null: 1); out [T, hidden].
 PL_API int pl_moe_down(const void* act, const void* down, const int32_t* ids, const float* weights, const void* also,
-                       void* out, int n_tokens, int hidden, int ff, int top, int n_experts, int dtype,
+                       const float* also_weights, void* out, int n_tokens, int hidden, int ff, int top, int n_experts, int dtype,
                        cudaStream_t stream) {
     PL_REQUIRE(n_tokens >= 0 && hidden > 0 && ff > 0 && top > 0 && n_experts > 0, "moe_down: bad sizes");
     const size_t smem = static_cast<size_t>(top) * ff * sizeof(float);
@@ -805,8 +836,8 @@ PL_API int pl_moe_down(const void* act, const void* down, const int32_t* ids, co
         }
         pl_launch_overlapped(moe_down_kernel<scalar_t>, grid, dim3(warps * 32), smem, stream,
                              static_cast<const scalar_t*>(act), static_cast<const scalar_t*>(down), ids, weights,
-                             static_cast<const scalar_t*>(also), static_cast<scalar_t*>(out), hidden, ff, top,
-                             n_experts, vectors);
+                             static_cast<const scalar_t*>(also), also_weights, static_cast<scalar_t*>(out), hidden, ff,
+                             top, n_experts, vectors);
     });
     PL_CHECK_LAUNCH("moe_down");
     return 0;
@@ -843,8 +874,8 @@ PL_API int pl_moe_gather(const void* x, int64_t x_stride, const int32_t* pair_of
     return 0;
 }
 
-PL_API int pl_moe_combine(const void* y, const int32_t* row_of_pair, const float* weights, const void* also, void* out,
-                          int n_tokens, int hidden, int top, int dtype, cudaStream_t stream) {
+PL_API int pl_moe_combine(const void* y, const int32_t* row_of_pair, const float* weights, const void* also,
+                          const float* also_weights, void* out, int n_tokens, int hidden, int top, int dtype, cudaStream_t stream) {
     PL_REQUIRE(n_tokens >= 0 && hidden > 0 && top > 0, "moe_combine: bad sizes");
     if (n_tokens == 0) {
         return 0;
@@ -854,7 +885,7 @@ PL_API int pl_moe_combine(const void* y, const int32_t* row_of_pair, const float
                                                  reinterpret_cast<uintptr_t>(out)) & 15) == 0;
         pl_launch_overlapped(moe_combine_kernel<scalar_t>, dim3(n_tokens), dim3(hidden >= 1024 ? 256 : 128), 0, stream,
                              static_cast<const scalar_t*>(y), row_of_pair, weights, static_cast<const scalar_t*>(also),
-                             static_cast<scalar_t*>(out), hidden, top, vectors);
+                             also_weights, static_cast<scalar_t*>(out), hidden, top, vectors);
     });
     PL_CHECK_LAUNCH("moe_combine");
     return 0;

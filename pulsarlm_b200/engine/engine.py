@@ -118,7 +118,7 @@ class Engine:
         self.runner = ModelRunner(self.model, self.cache)
         self.runner._bind()
         # Said once: a shape that the fast kernels do not take still runs, only slower.
-        notes = sorted({note for part in self.model.parts()
+        notes = sorted({note for part in self.model.all_parts()
                         for note in [getattr(part, "slow_path_note", lambda: None)()] if note})
         for note in notes:
             print(f"[pulsarlm_b200] note: {note}", file=sys.stderr, flush=True)

@@ -99,7 +99,7 @@ class ModelRunner:
         state_mixers = [self.model.cache_holder(key) for key in cache.state_layers]
         self.graphs_allowed = all(getattr(m, "captures_state_steps", lambda: False)() for m in state_mixers) and (
             cache.mass_decay is None or all(
-                getattr(part, "measures_mass_in_captured_steps", lambda: True)() for part in model.parts()))
+                getattr(part, "measures_mass_in_captured_steps", lambda: True)() for part in model.all_parts()))
         self.steps = 0
         self.tokens_run = 0
         self.graph_steps = 0

@@ -25,7 +25,7 @@ _PTR = ctypes.c_void_p
 _lib = None
 _lock = threading.Lock()
 
-ABI_VERSION = 28
+ABI_VERSION = 29
 
 DTYPE_CODE = {torch.float32: 0, torch.bfloat16: 1}
 
@@ -54,7 +54,7 @@ _SIGNATURES = {
                          _PTR, _I32, _I32, _I32, _I32, _I32, _I32, _PTR, _PTR, _F32, _PTR, _PTR],
     "pl_attention_simt": [_PTR, _I64, _PTR, _PTR, _I64, _I64, _I32, _I32, _PTR, _I32, _PTR, _PTR, _PTR, _I64,
                           _I32, _I32, _I32, _I32, _I32, _F32, _F32, _I32, _PTR, _PTR, _PTR, _PTR, _PTR, _I64, _PTR,
-                          _I32, _PTR, _PTR],
+                          _I32, _PTR, _PTR, _PTR],
     "pl_attention_decode": [_PTR, _I64, _PTR, _PTR, _I64, _I64, _I32, _I32, _PTR, _I32, _PTR, _PTR, _PTR, _I64,
                             _I32, _I32, _I32, _I32, _I32, _F32, _I32, _PTR, _PTR, _PTR, _PTR],
     "pl_attention_decode_mass": [_PTR, _I64, _PTR, _PTR, _I64, _I64, _I32, _I32, _PTR, _I32, _PTR, _PTR, _PTR, _I64,
@@ -77,6 +77,9 @@ _SIGNATURES = {
                                      _PTR, _I64, _I32, _I32, _I32, _I32, _F32, _I32, _PTR, _I32, _PTR, _PTR, _PTR],
     "pl_attention_prefill_tcgen05_bias": [_PTR, _I64, _I32, _PTR, _PTR, _I64, _I64, _I32, _I32, _PTR, _I32, _PTR, _I32,
                                           _PTR, _I64, _I32, _I32, _I32, _I32, _F32, _I32, _PTR, _PTR, _I32, _PTR, _PTR],
+    "pl_attention_prefill_tcgen05_slopes": [_PTR, _I64, _I32, _PTR, _PTR, _I64, _I64, _I32, _I32, _PTR, _I32, _PTR,
+                                            _I32, _PTR, _I64, _I32, _I32, _I32, _I32, _F32, _I32, _PTR, _PTR, _PTR,
+                                            _PTR, _PTR],
     "pl_attention_prefill_tcgen05_tile_rows": [_I32],
     "pl_attention_prefill_tcgen05_supports": [_I32, _I32, _I32, _I64, _I64, _I64, _I32],
     "pl_attention_prefill_tile_rows": [],
@@ -96,8 +99,8 @@ _SIGNATURES = {
     "pl_short_conv_state_strided": [_PTR, _I64, _PTR, _PTR, _PTR, _I32, _I32, _I32, _I32, _PTR],
     "pl_gated_delta": [_PTR, _PTR, _PTR, _I64, _PTR, _I64, _PTR, _I64, _PTR, _I64, _PTR, _PTR, _PTR, _PTR, _PTR, _PTR,
                        _PTR, _PTR, _PTR, _I64, _I32, _I32, _I32, _I32, _I32, _I32, _F32, _F32, _F32, _I32, _PTR],
-    "pl_moe_route": [_PTR, _I64, _PTR, _PTR, _PTR, _PTR, _I32, _I32, _I32, _I32, _I32, _I32, _I32, _I32, _I32, _I32,
-                     _PTR],
+    "pl_moe_route": [_PTR, _I64, _PTR, _PTR, _PTR, _PTR, _I32, _I32, _I32, _I32, _I32, _I32, _I32, _I32, _I32, _PTR,
+                     _I32, _PTR],
     "pl_moe_up": [_PTR, _I64, _PTR, _PTR, _PTR, _I32, _I32, _I32, _I32, _I32, _I32, _PTR],
     "pl_pair_embed": [_PTR, _PTR, _PTR, _PTR, _PTR, _PTR, _PTR, _PTR, _I32, _I32, _I32, _I32, _I64, _I64, _I32, _I32,
                       _PTR, _PTR],
@@ -105,13 +108,13 @@ _SIGNATURES = {
     "pl_norm_rope_mix_write": [_PTR, _PTR, _PTR, _I64, _PTR, _I64, _F32, _PTR, _PTR, _PTR, _PTR, _I32, _PTR, _PTR,
                                _I64, _I64, _I32, _I32, _PTR, _I32, _I32, _I32, _I32, _I32, _I32, _I32, _I32, _PTR,
                                _PTR, _F32, _I32, _PTR, _PTR],
-    "pl_moe_gate_up": [_PTR, _I64, _PTR, _PTR, _PTR, _I32, _I32, _I32, _I32, _I32, _I32, _PTR],
-    "pl_moe_down": [_PTR, _PTR, _PTR, _PTR, _PTR, _PTR, _I32, _I32, _I32, _I32, _I32, _I32, _PTR],
+    "pl_moe_gate_up": [_PTR, _I64, _PTR, _PTR, _PTR, _I32, _I32, _I32, _I32, _I32, _I32, _F32, _PTR, _I32, _PTR],
+    "pl_moe_down": [_PTR, _PTR, _PTR, _PTR, _PTR, _PTR, _PTR, _I32, _I32, _I32, _I32, _I32, _I32, _PTR],
     "pl_moe_sort": [_PTR, _I32, _I32, _PTR, _PTR, _PTR, _PTR],
     "pl_moe_gather": [_PTR, _I64, _PTR, _PTR, _I32, _I32, _I32, _I32, _PTR],
-    "pl_moe_combine": [_PTR, _PTR, _PTR, _PTR, _PTR, _I32, _I32, _I32, _I32, _PTR],
+    "pl_moe_combine": [_PTR, _PTR, _PTR, _PTR, _PTR, _PTR, _I32, _I32, _I32, _I32, _PTR],
     "pl_add_layernorm": [_PTR, _PTR, _PTR, _PTR, _F32, _PTR, _PTR, _PTR, _F32, _PTR, _I32, _I32, _I32, _I32, _PTR],
-    "pl_gated_act": [_PTR, _PTR, _I32, _I32, _I32, _I32, _PTR],
+    "pl_gated_act": [_PTR, _PTR, _I32, _I32, _I32, _F32, _PTR, _PTR, _I32, _PTR],
     "pl_sigmoid_gate": [_PTR, _I64, _PTR, _I64, _I32, _I32, _I32, _PTR],
     "pl_sigmoid_gate_heads": [_PTR, _I64, _PTR, _I64, _I32, _I32, _I32, _I32, _PTR],
     "pl_conv_norm_rope_write": [_PTR, _I64, _PTR, _PTR, _I32, _PTR, _PTR, _I32, _PTR, _PTR, _F32, _PTR, _I32, _I32, _F32,
@@ -119,6 +122,17 @@ _SIGNATURES = {
                                 _I32, _I32, _PTR, _PTR],
     "pl_latent_rope_write": [_PTR, _I64, _I32, _I32, _PTR, _I64, _PTR, _I64, _PTR, _F32, _I32, _I32, _PTR, _I32, _F32,
                              _PTR, _PTR, _PTR, _I32, _PTR, _I64, _I32, _I32, _I32, _I32, _PTR, _PTR],
+    "pl_side_norm": [_PTR, _PTR, _PTR, _PTR, _PTR, _PTR, _PTR, _F32, _F32, _PTR, _PTR, _F32, _PTR, _PTR, _PTR, _I32,
+                     _I32, _I32, _PTR],
+    "pl_conv_qkv_write": [_PTR, _I64, _PTR, _PTR, _I32, _PTR, _PTR, _I32, _I32, _F32, _I32, _PTR, _PTR, _PTR, _I32, _PTR,
+                          _PTR, _PTR, _I64, _I64, _I32, _I32, _I32, _I32, _I32, _I32, _I32, _I32, _I32, _I32, _I32, _PTR,
+                          _PTR],
+    "pl_ring_conv": [_PTR, _I64, _PTR, _PTR, _PTR, _I32, _PTR, _PTR, _PTR, _PTR, _PTR, _PTR, _I32, _I32, _I32, _PTR],
+    "pl_linear_scan": [_PTR, _PTR, _PTR, _PTR, _PTR, _PTR, _I64, _PTR, _PTR, _I64, _PTR, _I32, _PTR, _PTR, _PTR, _PTR,
+                       _PTR, _PTR, _I32, _I32, _I32, _I32, _I32, _I32, _PTR],
+    "pl_linear_step": [_PTR, _I64, _PTR, _PTR, _PTR, _I32, _PTR, _PTR, _PTR, _PTR, _PTR, _PTR, _I64, _PTR, _PTR, _PTR,
+                       _PTR, _PTR, _PTR, _I32, _I32, _I32, _PTR],
+    "pl_capped_scale": [_PTR, _I64, _F32, _F32, _PTR],
     "pl_sample": [_PTR, _I64, _I32, _I32, _PTR, _PTR, _PTR, _PTR, _PTR, _PTR, _PTR],
 }
 
@@ -588,22 +602,25 @@ def gated_delta(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, b_pre: torch.
 
 
 def moe_route(h: torch.Tensor, router: torch.Tensor, correction: torch.Tensor | None, top: int, n_groups: int,
-              keep: int, sigmoid_scores: bool = False, group_top: int = 1,
-              renormalise: bool = True) -> tuple[torch.Tensor, torch.Tensor]:
+              keep: int, sigmoid_scores: bool = False, group_top: int = 1, renormalise: bool = True,
+              shared_weights: torch.Tensor | None = None) -> tuple[torch.Tensor, torch.Tensor]:
     """(ids int32 [T, top], weights fp32 [T, top]) of the experts each token's router chooses (see csrc/moe.cu).
     sigmoid_scores: scores are sigmoids of the logits instead of their softmax; group_top: how many of a
-    group's largest choice scores add up to its score; renormalise: the chosen scores over their sum."""
-    _dev(h, router, correction)
+    group's largest choice scores add up to its score; renormalise: the chosen scores over their sum. shared_weights
+    (fp32 [T]): the router's last row is no expert's but a shared expert's gate, and its sigmoid goes there."""
+    _dev(h, router, correction, shared_weights)
     tokens, hidden = h.shape
-    n_experts = router.shape[0]
-    assert router.dtype == torch.float32 and router.shape == (n_experts, hidden) and router.is_contiguous()
+    n_experts = router.shape[0] - (1 if shared_weights is not None else 0)
+    assert router.dtype == torch.float32 and router.shape[1] == hidden and router.is_contiguous() and n_experts > 0
+    assert shared_weights is None or (shared_weights.dtype == torch.float32 and shared_weights.shape == (tokens,)
+                                      and shared_weights.is_contiguous())
     assert correction is None or (correction.dtype == torch.float32 and correction.shape == (n_experts,))
     assert h.stride(1) == 1
     ids = torch.empty((tokens, top), dtype=torch.int32, device=h.device)
     weights = torch.empty((tokens, top), dtype=torch.float32, device=h.device)
     _call("pl_moe_route", _p(h), h.stride(0) if tokens > 1 else hidden, _p(router), _p(correction), _p(ids),
           _p(weights), tokens, hidden, n_experts, top, n_groups, keep, int(bool(sigmoid_scores)), int(group_top),
-          int(bool(renormalise)), _code(h.dtype), _stream())
+          int(bool(renormalise)), _p(shared_weights), _code(h.dtype), _stream())
     return ids, weights
 
 
@@ -619,30 +636,37 @@ def moe_up(h: torch.Tensor, up: torch.Tensor, ids: torch.Tensor, act: torch.Tens
           n_experts, _code(h.dtype), _stream())
 
 
-def moe_gate_up(h: torch.Tensor, gate_up: torch.Tensor, ids: torch.Tensor, act: torch.Tensor) -> None:
-    """act[t * top + j] = silu(Wg h_t) * (Wu h_t) with the weights of expert ids[t, j]; gate_up [E, 2 * ff, H]."""
-    _dev(h, gate_up, ids, act)
+def moe_gate_up(h: torch.Tensor, gate_up: torch.Tensor, ids: torch.Tensor, act: torch.Tensor,
+                limit: float | None = None, in_weights: torch.Tensor | None = None) -> None:
+    """act[t * top + j] = silu(Wg h_t) * (Wu h_t) with the weights of expert ids[t, j]; gate_up [E, 2 * ff, H]. With
+    `limit`: the clamped unit (see csrc/gate_units.cuh) of w Wg h_t and w Wu h_t, w = in_weights[t, j] (fp32; None: 1)."""
+    _dev(h, gate_up, ids, act, in_weights)
+    assert in_weights is None or (limit is not None and in_weights.dtype == torch.float32 and in_weights.is_contiguous()
+                                  and in_weights.shape == ids.shape)
     tokens, hidden = h.shape
     n_experts, two_ff, _ = gate_up.shape
     top = ids.shape[1]
     assert gate_up.is_contiguous() and gate_up.shape[2] == hidden and gate_up.dtype == h.dtype == act.dtype
     assert act.is_contiguous() and act.shape == (tokens * top, two_ff // 2) and ids.is_contiguous() and h.stride(1) == 1
     _call("pl_moe_gate_up", _p(h), h.stride(0) if tokens > 1 else hidden, _p(gate_up), _p(ids), _p(act), tokens,
-          hidden, two_ff // 2, top, n_experts, _code(h.dtype), _stream())
+          hidden, two_ff // 2, top, n_experts, int(limit is not None), float(limit or 0.0), _p(in_weights),
+          _code(h.dtype), _stream())
 
 
-def moe_down(act: torch.Tensor, down: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor,
-             also: torch.Tensor | None, out: torch.Tensor) -> None:
-    """out[t] = sum_j weights[t, j] * W_down,ids[t, j] act[t * top + j] + also[t]; down [E, H, ff]."""
-    _dev(act, down, ids, weights, also, out)
+def moe_down(act: torch.Tensor, down: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor | None,
+             also: torch.Tensor | None, out: torch.Tensor, also_weights: torch.Tensor | None = None) -> None:
+    """out[t] = sum_j weights[t, j] * W_down,ids[t, j] act[t * top + j] + also_weights[t] * also[t]; down [E, H, ff];
+    weights None: all 1; also_weights (fp32 [T]) None: 1."""
+    _dev(act, down, ids, weights, also, out, also_weights)
+    assert also_weights is None or (also_weights.dtype == torch.float32 and also_weights.shape == (out.shape[0],))
     tokens, hidden = out.shape
     n_experts, _, ff = down.shape
     top = ids.shape[1]
     assert down.is_contiguous() and down.shape[1] == hidden and down.dtype == act.dtype == out.dtype
     assert act.is_contiguous() and act.shape == (tokens * top, ff) and out.is_contiguous()
-    assert weights.dtype == torch.float32 and weights.is_contiguous() and weights.shape == ids.shape
+    assert weights is None or (weights.dtype == torch.float32 and weights.is_contiguous() and weights.shape == ids.shape)
     assert also is None or (also.shape == out.shape and also.is_contiguous() and also.dtype == out.dtype)
-    _call("pl_moe_down", _p(act), _p(down), _p(ids), _p(weights), _p(also), _p(out), tokens, hidden, ff, top,
+    _call("pl_moe_down", _p(act), _p(down), _p(ids), _p(weights), _p(also), _p(also_weights), _p(out), tokens, hidden, ff, top,
           n_experts, _code(out.dtype), _stream())
 
 
@@ -670,16 +694,18 @@ def moe_gather(x: torch.Tensor, pair_of_row: torch.Tensor, top: int) -> torch.Te
     return out
 
 
-def moe_combine(y: torch.Tensor, row_of_pair: torch.Tensor, weights: torch.Tensor, also: torch.Tensor | None,
-                out: torch.Tensor) -> None:
-    """out[t] = sum_j weights[t, j] * y[row_of_pair[t * top + j]] + also[t]."""
-    _dev(y, row_of_pair, weights, also, out)
+def moe_combine(y: torch.Tensor, row_of_pair: torch.Tensor, weights: torch.Tensor | None, also: torch.Tensor | None,
+                out: torch.Tensor, also_weights: torch.Tensor | None = None) -> None:
+    """out[t] = sum_j weights[t, j] * y[row_of_pair[t * top + j]] + also_weights[t] * also[t]; weights None: all 1;
+    also_weights (fp32 [T]) None: 1."""
+    _dev(y, row_of_pair, weights, also, out, also_weights)
     tokens, hidden = out.shape
-    top = weights.shape[1]
+    top = y.shape[0] // max(tokens, 1)
+    assert also_weights is None or (also_weights.dtype == torch.float32 and also_weights.shape == (tokens,))
     assert y.is_contiguous() and y.shape == (tokens * top, hidden) and y.dtype == out.dtype and out.is_contiguous()
-    assert weights.dtype == torch.float32 and weights.is_contiguous()
+    assert weights is None or (weights.dtype == torch.float32 and weights.is_contiguous() and weights.shape == (tokens, top))
     assert also is None or (also.shape == out.shape and also.is_contiguous() and also.dtype == out.dtype)
-    _call("pl_moe_combine", _p(y), _p(row_of_pair), _p(weights), _p(also), _p(out), tokens, hidden, top,
+    _call("pl_moe_combine", _p(y), _p(row_of_pair), _p(weights), _p(also), _p(also_weights), _p(out), tokens, hidden, top,
           _code(out.dtype), _stream())
 
 
@@ -726,16 +752,23 @@ def add_layernorm(x: torch.Tensor, y: torch.Tensor | None, y_weight: torch.Tenso
           float(eps), _p(rows), n_rows, hidden, int(weight is not None), _code(dtype), _stream())
 
 
-GATED_ACT = {"silu": 0, "gelu_tanh": 1}
+GATED_ACT = {"silu": 0, "gelu_tanh": 1, "clamped": 2}
 
 
-def gated_act(gate_up: torch.Tensor, out: torch.Tensor, act: str) -> None:
-    """out[t, i] = act(gate_up[t, i]) * gate_up[t, I + i]; act "silu" or "gelu_tanh" (the tanh form)."""
-    _dev(gate_up, out)
+def gated_act(gate_up: torch.Tensor, out: torch.Tensor, act: str, limit: float = 0.0,
+              row_weights: torch.Tensor | None = None, row_index: torch.Tensor | None = None) -> None:
+    """out[t, i] = act(gate_up[t, i]) * gate_up[t, I + i]; act "silu" or "gelu_tanh" (the tanh form). "clamped": g =
+    min(w gate_up[t, i], limit), u = clamp(w gate_up[t, I + i], -limit, limit), out = g sigmoid(1.702 g) (u + 1), w the
+    row's weight: row_weights (fp32) at row_index[t] (int32; None: at t), 1 without."""
+    _dev(gate_up, out, row_weights, row_index)
+    if row_weights is not None:
+        assert row_weights.dtype == torch.float32 and row_weights.is_contiguous()
+        assert row_index is None or (row_index.dtype == torch.int32 and row_index.numel() == gate_up.shape[0])
     tokens, two_i = gate_up.shape
     assert two_i % 2 == 0 and out.shape == (tokens, two_i // 2) and out.dtype == gate_up.dtype
     assert gate_up.is_contiguous() and out.is_contiguous()
-    _call("pl_gated_act", _p(gate_up), _p(out), tokens, two_i // 2, GATED_ACT[act], _code(out.dtype), _stream())
+    _call("pl_gated_act", _p(gate_up), _p(out), tokens, two_i // 2, GATED_ACT[act], float(limit), _p(row_weights),
+          _p(row_index), _code(out.dtype), _stream())
 
 
 def sigmoid_gate(x: torch.Tensor, gate: torch.Tensor) -> None:
@@ -826,6 +859,142 @@ def latent_rope_write(q: torch.Tensor, q_out: torch.Tensor, z: torch.Tensor | No
           z.stride(0) if z is not None else 0, _p(weight), float(eps), rank, rot, _p(inv_freq),
           int(bool(interleaved)), float(amplitude), _p(pos), _p(entry), _p(table), table.shape[1], _p(pool),
           pool.stride(0), page_size, pool.shape[0], tokens, _code(q.dtype), _p(status), _stream())
+
+
+def side_norm(x: torch.Tensor, sides: tuple | None, factor: float, y_eps: float, y3: torch.Tensor | None,
+              weight: torch.Tensor | None, eps: float, out: torch.Tensor | None, rows: torch.Tensor | None = None,
+              entered: torch.Tensor | None = None) -> None:
+    """x fp32 [T, H] += factor * (rmsnorm(y1 + b1) * w1 + rmsnorm(y2 + b2) * w2) + y3 (in place unless rows is given),
+    sides = (y1, b1, w1, y2, b2, w2) or None; then out = rmsnorm(x) * weight, or with `entered` (fp32 [T, H]) out [T,
+    2 H] = [x, entered]. y1, y2, y3 and out in the engine's dtype, biases (or None) and weights fp32. With rows (int32
+    [R]) output row r is made from source row rows[r] and x is left as it was. out None: the stream alone."""
+    y1, b1, w1, y2, b2, w2 = sides if sides is not None else (None,) * 6
+    _dev(x, y1, b1, w1, y2, b2, w2, y3, weight, out, rows, entered)
+    assert x.dtype == torch.float32 and x.is_contiguous()
+    hidden = x.shape[-1]
+    dtype = next((t.dtype for t in (out, y1, y3) if t is not None), torch.float32)
+    for y in (y1, y2, y3):
+        assert y is None or (y.shape == x.shape and y.dtype == dtype and y.is_contiguous())
+    for v in (b1, w1, b2, w2, weight):
+        assert v is None or (v.dtype == torch.float32 and v.shape == (hidden,) and v.is_contiguous())
+    assert rows is None or (rows.dtype == torch.int32 and rows.is_contiguous())
+    n_rows = rows.numel() if rows is not None else x.shape[0]
+    if entered is not None:
+        assert entered.dtype == torch.float32 and entered.shape == x.shape and entered.is_contiguous()
+    if out is not None:
+        assert out.is_contiguous() and out.shape == (n_rows, hidden * (2 if entered is not None else 1))
+        assert out.dtype == dtype
+    _call("pl_side_norm", _p(x), _p(y1), _p(b1), _p(w1), _p(y2), _p(b2), _p(w2), float(factor), float(y_eps), _p(y3),
+          _p(weight), float(eps), _p(entered), _p(out), _p(rows), n_rows, hidden, _code(dtype), _stream())
+
+
+def conv_qkv_write(proj: torch.Tensor, row_stride: int, bias: torch.Tensor | None, weight: torch.Tensor,
+                   state: torch.Tensor | None, slots: torch.Tensor, update_state: bool, temp_coef: float, temp_every: int,
+                   pos: torch.Tensor, entry: torch.Tensor, table: torch.Tensor, q_out: torch.Tensor, k_pool: torch.Tensor,
+                   v_pool: torch.Tensor, page_size: int, n_kv: int, dim: int, vdim: int, k_col: int, v_col: int,
+                   status: torch.Tensor | None = None) -> None:
+    """From a token's projected q, k and v channels (proj [T, channels], columns of a wider matrix whose rows are
+    `row_stride` elements apart; k from column k_col, v from v_col) to q_out [T, nh, row] and the token's page: bias,
+    causal convolution over time (weight fp32 [taps, channels], state [slots, taps - 1, channels] the projected rows
+    before this step's), the query's temperature 1 + temp_coef * ln(floor((pos + 1) / temp_every) + 1) (temp_coef 0:
+    none), rows of a common size with zeros past dim (q, k) and vdim (v). update_state: every entry brings one token
+    and its slot moves on in the same launch."""
+    _dev(proj, bias, weight, state, slots, pos, entry, table, q_out, k_pool, v_pool, status)
+    tokens, channels = proj.shape
+    n_heads, row = q_out.shape[1], q_out.shape[2]
+    taps = weight.shape[0]
+    assert proj.stride(1) == 1 and (tokens == 1 or proj.stride(0) == row_stride)
+    assert weight.dtype == torch.float32 and weight.shape == (taps, channels) and weight.is_contiguous()
+    assert bias is None or (bias.dtype == torch.float32 and bias.shape == (channels,) and bias.is_contiguous())
+    if taps > 1:
+        assert state.dtype == proj.dtype and state.is_contiguous() and state.shape[1:] == (taps - 1, channels)
+    assert q_out.shape[0] == tokens and q_out.is_contiguous() and q_out.dtype == proj.dtype == k_pool.dtype == v_pool.dtype
+    n_pages = k_pool.shape[0]
+    assert k_pool.shape == (n_pages, n_kv, page_size, row) == v_pool.shape and k_pool.stride() == v_pool.stride()
+    assert k_pool.stride(3) == 1 and k_pool.stride(2) == row and table.dim() == 2 and table.is_contiguous()
+    for t in (pos, entry, table, slots):
+        assert t.dtype == torch.int32
+    _call("pl_conv_qkv_write", _p(proj), int(row_stride), _p(bias), _p(weight), taps, _p(state) if taps > 1 else None,
+          _p(slots), channels, int(bool(update_state)), float(temp_coef), int(temp_every), _p(pos), _p(entry), _p(table),
+          table.shape[1], _p(q_out), _p(k_pool), _p(v_pool), k_pool.stride(0), k_pool.stride(1), page_size, n_pages, tokens,
+          n_heads, n_kv, dim, vdim, row, k_col, v_col, _code(proj.dtype), _p(status), _stream())
+
+
+def ring_conv(x: torch.Tensor, row_stride: int, x_bias: torch.Tensor, weight: torch.Tensor, conv_bias: torch.Tensor,
+              ring: torch.Tensor, first: torch.Tensor, entry: torch.Tensor, slots: torch.Tensor, pos: torch.Tensor,
+              out: torch.Tensor) -> None:
+    """out [T, R] = conv_bias + sum_j weight[j] * (x[t - (taps - 1) + j] + x_bias) along each sequence, zeros before
+    position 0. x [T, R] columns of a matrix whose rows are `row_stride` elements apart; weight fp32 [taps, R]; ring
+    [slots, taps, R] the inputs of earlier steps, position p in row p mod taps (read only); first int32 [entries]."""
+    _dev(x, x_bias, weight, conv_bias, ring, first, entry, slots, pos, out)
+    tokens, width = x.shape
+    taps = weight.shape[0]
+    assert x.stride(1) == 1 and (tokens == 1 or x.stride(0) == row_stride) and out.shape == x.shape and out.is_contiguous()
+    assert ring.is_contiguous() and ring.shape[1:] == (taps, width) and ring.dtype == x.dtype == out.dtype
+    for v, shape in ((weight, (taps, width)), (x_bias, (width,)), (conv_bias, (width,))):
+        assert v.dtype == torch.float32 and v.shape == shape and v.is_contiguous()
+    for t in (first, entry, slots, pos):
+        assert t.dtype == torch.int32 and t.is_contiguous()
+    _call("pl_ring_conv", _p(x), int(row_stride), _p(x_bias), _p(weight), _p(conv_bias), taps, _p(ring), _p(first), _p(entry),
+          _p(slots), _p(pos), _p(out), tokens, width, _code(x.dtype), _stream())
+
+
+def linear_scan(pre: torch.Tensor, ra_bias: torch.Tensor, ri_bias: torch.Tensor, decay: torch.Tensor, u: torch.Tensor,
+                y: torch.Tensor, y_bias: torch.Tensor, x: torch.Tensor, row_stride: int, ring: torch.Tensor,
+                states: torch.Tensor, first: torch.Tensor, count: torch.Tensor, slots: torch.Tensor, pos: torch.Tensor,
+                longest: int, out: torch.Tensor) -> None:
+    """The gated linear recurrence over every entry's rows (see csrc/linear_recurrence.cu): pre fp32 [blocks, T, 2 *
+    block] the gates' products, u [T, R], y and x [T, R] columns of one matrix (`row_stride`), states fp32 [slots, R]
+    and the ring [slots, taps, R] move on; out [T, R] = S * gelu(y + y_bias)."""
+    _dev(pre, ra_bias, ri_bias, decay, u, y, y_bias, x, ring, states, first, count, slots, pos, out)
+    tokens, width = u.shape
+    blocks, block = pre.shape[0], pre.shape[2] // 2
+    assert pre.dtype == torch.float32 and pre.is_contiguous() and pre.shape[1] == tokens and blocks * block == width
+    assert u.is_contiguous() and out.is_contiguous() and out.shape == u.shape and x.shape == y.shape == u.shape
+    for t in (x, y):
+        assert t.stride(1) == 1 and (tokens == 1 or t.stride(0) == row_stride) and t.dtype == u.dtype == out.dtype
+    assert states.dtype == torch.float32 and states.is_contiguous() and states.shape[1:] == (width,)
+    assert ring.is_contiguous() and ring.shape[2] == width and ring.dtype == u.dtype
+    for v in (ra_bias, ri_bias, decay, y_bias):
+        assert v.dtype == torch.float32 and v.shape == (width,) and v.is_contiguous()
+    for t in (first, count, slots, pos):
+        assert t.dtype == torch.int32 and t.is_contiguous()
+    _call("pl_linear_scan", _p(pre), _p(ra_bias), _p(ri_bias), _p(decay), _p(u), _p(y), int(row_stride), _p(y_bias), _p(x),
+          int(row_stride), _p(ring), ring.shape[1], _p(states), _p(first), _p(count), _p(slots), _p(pos), _p(out), tokens,
+          first.numel(), int(longest), width, block, _code(u.dtype), _stream())
+
+
+def linear_step(x: torch.Tensor, row_stride: int, x_bias: torch.Tensor, weight: torch.Tensor, conv_bias: torch.Tensor,
+                ring: torch.Tensor, gates: torch.Tensor, ra_bias: torch.Tensor, ri_bias: torch.Tensor, decay: torch.Tensor,
+                y: torch.Tensor, y_bias: torch.Tensor, states: torch.Tensor, entry: torch.Tensor, slots: torch.Tensor,
+                pos: torch.Tensor, out: torch.Tensor) -> None:
+    """ring_conv, the gates' products and linear_scan for a step in which every entry brings one token, bfloat16, in
+    one launch. gates [blocks, 2 * block, block]."""
+    _dev(x, x_bias, weight, conv_bias, ring, gates, ra_bias, ri_bias, decay, y, y_bias, states, entry, slots, pos, out)
+    tokens, width = x.shape
+    blocks, two_block, block = gates.shape
+    taps = weight.shape[0]
+    assert x.dtype == torch.bfloat16 == y.dtype == gates.dtype == ring.dtype == out.dtype
+    assert two_block == 2 * block and blocks * block == width and gates.is_contiguous()
+    for t in (x, y):
+        assert t.shape == (tokens, width) and t.stride(1) == 1 and (tokens == 1 or t.stride(0) == row_stride)
+    assert out.shape == x.shape and out.is_contiguous() and ring.is_contiguous() and ring.shape[1:] == (taps, width)
+    assert states.dtype == torch.float32 and states.is_contiguous() and states.shape[1:] == (width,)
+    for v, shape in ((weight, (taps, width)), (x_bias, (width,)), (conv_bias, (width,)), (ra_bias, (width,)),
+                     (ri_bias, (width,)), (decay, (width,)), (y_bias, (width,))):
+        assert v.dtype == torch.float32 and v.shape == shape and v.is_contiguous()
+    for t in (entry, slots, pos):
+        assert t.dtype == torch.int32 and t.is_contiguous()
+    _call("pl_linear_step", _p(x), int(row_stride), _p(x_bias), _p(weight), _p(conv_bias), taps, _p(ring), _p(gates),
+          _p(ra_bias), _p(ri_bias), _p(decay), _p(y), int(row_stride), _p(y_bias), _p(states), _p(entry), _p(slots), _p(pos),
+          _p(out), tokens, width, block, _stream())
+
+
+def capped_scale(x: torch.Tensor, scale: float, cap: float) -> None:
+    """x (fp32, contiguous) = cap * tanh(x * scale / cap), in place."""
+    _dev(x)
+    assert x.dtype == torch.float32 and x.is_contiguous()
+    _call("pl_capped_scale", _p(x), x.numel(), float(scale), float(cap), _stream())
 
 
 def swiglu(gate_up: torch.Tensor, out: torch.Tensor) -> None:
@@ -986,7 +1155,7 @@ def attention_simt(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, 
                    scale: float, status: torch.Tensor | None = None, mass_sum: torch.Tensor | None = None,
                    weight_sum: torch.Tensor | None = None, query_weights: torch.Tensor | None = None,
                    softcap: float = 0.0, sinks: torch.Tensor | None = None, gate: torch.Tensor | None = None,
-                   distance_bias: torch.Tensor | None = None) -> None:
+                   distance_bias: torch.Tensor | None = None, distance_slopes: torch.Tensor | None = None) -> None:
     """Causal paged attention; q and out [T, nh, hd] (row strides free), pools
     [pages, nkv, page_size, hd]. With mass_sum fp32 [pages, nh] and weight_sum fp32
     [pages], the attention mass of every attended page is added to them
@@ -995,9 +1164,13 @@ def attention_simt(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, 
     h's softmax denominator (a term with no key and no value). gate [T, nh] logits (row
     stride free): head h's output for token t is multiplied by sigmoid(gate[t, h]). distance_bias
     fp32 [nh, rows]: entry min(distance, rows - 1) of a head's row is added to its scaled scores of a
-    key `distance` tokens before the query."""
+    key `distance` tokens before the query. distance_slopes fp32 [nh]: slopes[h] * distance is taken off head h's
+    scaled scores."""
     _dev(q, k_pool, v_pool, table, pos, entry, out, status, mass_sum, weight_sum, query_weights, sinks, gate,
-         distance_bias)
+         distance_bias, distance_slopes)
+    if distance_slopes is not None:
+        assert distance_slopes.dtype == torch.float32 and distance_slopes.shape == (q.shape[1],)
+        assert distance_slopes.is_contiguous()
     if distance_bias is not None:
         assert distance_bias.dtype == torch.float32 and distance_bias.dim() == 2 and distance_bias.is_contiguous()
         assert distance_bias.shape[0] == q.shape[1] and distance_bias.shape[1] > 0
@@ -1025,7 +1198,7 @@ def attention_simt(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, 
           n_heads, n_kv, head_dim, int(window or 0), float(scale), float(softcap or 0.0), _code(q.dtype),
           _p(mass_sum), _p(weight_sum), _p(query_weights), _p(sinks), _p(gate),
           gate.stride(0) if gate is not None else 0, _p(distance_bias),
-          distance_bias.shape[1] if distance_bias is not None else 0, _p(status), _stream())
+          distance_bias.shape[1] if distance_bias is not None else 0, _p(distance_slopes), _p(status), _stream())
 
 
 def attention_decode_supports(head_dim: int, group: int, page_size: int, dtype: torch.dtype) -> bool:
@@ -1114,22 +1287,27 @@ def attention_decode_ctas_per_sm(head_dim: int) -> int:
 
 class _AttentionExtras(ctypes.Structure):
     _fields_ = [("sinks", _PTR), ("gate", _PTR), ("gate_row_stride", _I64), ("split_weights", _I32),
-                ("softcap", _F32), ("distance_bias", _PTR), ("bias_rows", _I32)]
+                ("softcap", _F32), ("distance_bias", _PTR), ("bias_rows", _I32), ("distance_slopes", _PTR)]
 
 
 def attention_extras(q: torch.Tensor, sinks: torch.Tensor | None, gate: torch.Tensor | None,
-                     split_weights: bool, softcap: float = 0.0,
-                     distance_bias: torch.Tensor | None = None) -> "_AttentionExtras | None":
+                     split_weights: bool, softcap: float = 0.0, distance_bias: torch.Tensor | None = None,
+                     distance_slopes: torch.Tensor | None = None) -> "_AttentionExtras | None":
     """What the tensor-core attention kernels take beyond plain softmax attention (the struct
     PlAttentionExtras): sinks fp32 [nh] (exp(sinks[h]) joins head h's denominator), gate [T, nh]
     logits in q's dtype (outputs times their sigmoid), split_weights (softmax weights enter the
     value product as two bfloat16 terms), softcap (> 0: scaled scores pass through softcap *
     tanh(s / softcap)), distance_bias fp32 [nh, rows] (entry min(distance, rows - 1) of a head's row joins
-    its scaled scores of a key `distance` tokens before the query). None when nothing is asked for. The tensors
-    must outlive the call that takes the struct."""
-    if sinks is None and gate is None and not split_weights and not softcap and distance_bias is None:
+    its scaled scores of a key `distance` tokens before the query), distance_slopes fp32 [nh] (slopes[h] * distance
+    is taken off head h's scaled scores). None when nothing is asked for. The tensors must outlive the call that takes
+    the struct."""
+    if sinks is None and gate is None and not split_weights and not softcap and distance_bias is None \
+            and distance_slopes is None:
         return None
-    _dev(sinks, gate, distance_bias)
+    _dev(sinks, gate, distance_bias, distance_slopes)
+    if distance_slopes is not None:
+        assert distance_slopes.dtype == torch.float32 and distance_slopes.shape == (q.shape[1],)
+        assert distance_slopes.is_contiguous()
     if distance_bias is not None:
         assert distance_bias.dtype == torch.float32 and distance_bias.dim() == 2 and distance_bias.is_contiguous()
         assert distance_bias.shape[0] == q.shape[1] and distance_bias.shape[1] > 0
@@ -1139,7 +1317,7 @@ def attention_extras(q: torch.Tensor, sinks: torch.Tensor | None, gate: torch.Te
         assert gate.dtype == q.dtype and gate.shape == (q.shape[0], q.shape[1]) and gate.stride(1) == 1
     return _AttentionExtras(_p(sinks), _p(gate), gate.stride(0) if gate is not None else 0, int(bool(split_weights)),
                             float(softcap or 0.0), _p(distance_bias),
-                            distance_bias.shape[1] if distance_bias is not None else 0)
+                            distance_bias.shape[1] if distance_bias is not None else 0, _p(distance_slopes))
 
 
 def attention_decode(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, table: torch.Tensor,
@@ -1268,9 +1446,12 @@ def attention_prefill_tcgen05(q: torch.Tensor, k_pool: torch.Tensor, v_pool: tor
                               tiles: torch.Tensor, out: torch.Tensor, page_size: int, window: int | None,
                               scale: float, status: torch.Tensor | None = None, n_splits: int = 1,
                               scratch: torch.Tensor | None = None, wide: bool = False,
-                              mass: tuple | None = None, distance_bias: torch.Tensor | None = None) -> None:
+                              mass: tuple | None = None, distance_bias: torch.Tensor | None = None,
+                              distance_slopes: torch.Tensor | None = None, sinks: torch.Tensor | None = None) -> None:
     """As attention_prefill, on the tcgen05 tensor cores. `distance_bias` fp32 [nh, rows] (even GQA groups, no
-    wide tiles, no mass): entry min(distance, rows - 1) of a head's row joins its scaled scores. With n_splits > 1 every tile's
+    wide tiles, no mass): entry min(distance, rows - 1) of a head's row joins its scaled scores. `distance_slopes` fp32
+    [nh] (no mass; an odd group takes narrow and wide tiles alike): slopes[h] * distance is taken off head h's scaled
+    scores, and `sinks` fp32 [nh], with slopes only, join the denominators as exp(sinks[h]). With n_splits > 1 every tile's
     keys are shared out over that many CTAs and merged through `scratch` (float32,
     attention_prefill_scratch_floats elements): for few tiles over many keys. `wide`: the
     tiles have up to attention_prefill_tcgen05_tile_rows(group) rows instead of 128.
@@ -1304,6 +1485,17 @@ def attention_prefill_tcgen05(q: torch.Tensor, k_pool: torch.Tensor, v_pool: tor
     assert k_pool.stride() == v_pool.stride() and k_pool.stride(3) == 1 and k_pool.stride(2) == head_dim
     assert table.dtype == torch.int32 and table.dim() == 2 and table.is_contiguous()
     assert tiles.dtype == torch.int32 and tiles.dim() == 2 and tiles.shape[1] == 4 and tiles.is_contiguous()
+    if distance_slopes is not None:
+        _dev(distance_slopes, sinks)
+        assert mass is None and distance_bias is None
+        for v in (distance_slopes, sinks):
+            assert v is None or (v.dtype == torch.float32 and v.shape == (n_heads,) and v.is_contiguous())
+        _call("pl_attention_prefill_tcgen05_slopes", _p(q), q.stride(0), tokens, _p(k_pool), _p(v_pool), k_pool.stride(0),
+              k_pool.stride(1), page_size, n_pages, _p(table), table.shape[1], _p(tiles), tiles.shape[0], _p(out),
+              out.stride(0), n_heads, n_kv, head_dim, int(window or 0), float(scale), int(n_splits), _p(scratch),
+              _p(distance_slopes), _p(sinks), _p(status), _stream())
+        return
+    assert sinks is None
     if distance_bias is not None:
         _dev(distance_bias)
         assert mass is None and not wide and (n_heads // n_kv) % 2 == 0

@@ -85,6 +85,8 @@ def _all_part_specs(spec: ModelSpec):
     yield "embedding", spec.embedding
     for layer in spec.layers:
         yield from part_class("block", layer.block).part_specs(layer)
+    if spec.join is not None:
+        yield "join", spec.join
     yield "norm", spec.final_norm
     yield "head", spec.head
 
@@ -116,6 +118,7 @@ class Model:
         self.blocks = [part_class("block", layer.block)(layer, self.ctx) for layer in spec.layers]
         self.final_norm = build_part("norm", spec.final_norm, self.ctx)
         self.head = build_part("head", spec.head, self.ctx)
+        self.join = build_part("join", spec.join, self.ctx) if spec.join is not None else None
         self.loaded = False
         # The cache units, in the order the cache manager hears of them: one per layer, or
         # (spec.cache_per_run) one per entry of the order. `_unit_layer[u]` is the layer of unit u.
@@ -128,6 +131,9 @@ class Model:
         for r in self._rejoin:
             if not 0 < r < len(spec.order):
                 raise ValueError(f"the embedding cannot rejoin the stream before run {r} of {len(spec.order)}")
+        self._join_runs = frozenset(int(r) for r in spec.join_runs)
+        if self._join_runs and (self.join is None or not all(0 <= r < len(spec.order) for r in self._join_runs)):
+            raise ValueError(f"the stream cannot be joined before the runs {sorted(self._join_runs)} of {len(spec.order)}")
 
     # ------------------------------------------------------------------ weights
     def tensor_needs(self) -> dict[str, TensorNeed]:
@@ -137,8 +143,16 @@ class Model:
         yield self.embedding
         for b in self.blocks:
             yield from b.parts()
+        if self.join is not None:
+            yield self.join
         yield self.final_norm
         yield self.head
+
+    def all_parts(self):
+        """Every part, those inside other parts (`inner_parts()`, loaded by their owners) included."""
+        for part in self.parts():
+            yield part
+            yield from getattr(part, "inner_parts", lambda: [])()
 
     def load(self, tensors: dict[str, torch.Tensor]) -> None:
         """`tensors`: checked, converted, on the device (see weights.loader)."""
@@ -200,7 +214,7 @@ class Model:
     def planners(self) -> list:
         """The parts that plan steps on the host, one per distinct plan_key()."""
         seen: dict = {}
-        for part in self.parts():
+        for part in self.all_parts():
             key_of = getattr(part, "plan_key", None)
             key = key_of() if key_of is not None else None
             if key is not None and key not in seen:
@@ -263,7 +277,7 @@ class Model:
             raise RuntimeError("the model has no weights loaded")
         x = self.embedding.forward(batch.tokens, batch)
         delta = None
-        entered = x.clone() if self._rejoin else None  # (the stream is updated in place)
+        entered = x.clone() if self._rejoin or self._join_runs else None  # (the stream is updated in place)
         repeated = self._run_bindings is not None and len(self.spec.order) != len(set(self.spec.order))
         for run, index in enumerate(self.spec.order):
             block = self.blocks[index]
@@ -271,6 +285,8 @@ class Model:
                 self._bind_block(block, self._run_bindings[run])
             if run in self._rejoin:
                 x, delta = self._rejoin_stream(x, delta, entered)
+            if run in self._join_runs:
+                x, delta = self.join.forward(x, delta, entered), None
             x, delta = block.forward(x, delta, batch)
         if batch.want_rows is None or batch.want_rows.numel() == 0:
             return None

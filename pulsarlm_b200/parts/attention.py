@@ -242,6 +242,8 @@ class Attention(Part):
         # fp32 [n_heads, rows], set by a mixer that has one: entry min(distance, rows - 1) of a head's row joins
         # its scaled scores of a key `distance` tokens before the query
         self.distance_bias: torch.Tensor | None = None
+        # fp32 [n_heads], set by a mixer that has them: slope * distance is taken off a head's scaled scores
+        self.distance_slopes: torch.Tensor | None = None
         self.head_gate = False  # (a mixer that multiplies every head's output by a sigmoid hands `attend` the logits)
         # Whether the tensor-core kernels' build with extras feeds the softmax weights to the value product as two
         # bfloat16 terms (16 mantissa bits) or as one (8, as the plain build does; a third less tensor-core work).
@@ -444,10 +446,11 @@ class Attention(Part):
         return self._kernels(self.ctx.dtype)[0]
 
     def _wants_extras(self) -> bool:
-        """A score cap, a sink term, a bias by distance or a gate per head: the tensor-core kernels
-        take them in their build with extras (csrc/attention_decode.cu, attention_prefill.cu),
-        without work lists, wide tiles or attention mass."""
-        return bool(self.softcap) or self.sinks is not None or self.distance_bias is not None or self.head_gate
+        """A score cap, a sink term, a bias by distance (a table or slopes) or a gate per head: the
+        tensor-core kernels take them in their build with extras (csrc/attention_decode.cu,
+        attention_prefill.cu), without work lists or attention mass."""
+        return (bool(self.softcap) or self.sinks is not None or self.distance_bias is not None or self.head_gate
+                or self.distance_slopes is not None)
 
     def plan_key(self):
         """Layers of equal tiling share one plan: the tile lists depend on the kernels'
@@ -456,7 +459,7 @@ class Attention(Part):
             return None
         wide = (self.n_heads // self.n_kv) % 2 == 1
         return ("attention", self.cache.page_size, self.head_dim, self.n_heads // self.n_kv, wide,
-                self.ctx.dtype, self._wants_extras(), self.n_kv, self.window)
+                self.ctx.dtype, self._wants_extras(), self.distance_slopes is not None, self.n_kv, self.window)
 
     def native_key(self):
         """What `native_choice` depends on beyond `plan_key`: layers that agree in both get
@@ -532,7 +535,7 @@ class Attention(Part):
             start = step.context_lens[e] - n
             for r in range(0, n, rows):
                 tiles.append((at + r, min(rows, n - r), start + r, e))
-            if wide_rows > rows and not extras:
+            if wide_rows > rows and (not extras or self.distance_slopes is not None):
                 for r in range(0, n, wide_rows):
                     wide_tiles.append((at + r, min(wide_rows, n - r), start + r, e))
         tiles.sort(key=lambda t: -(t[2] + t[1]))
@@ -548,6 +551,12 @@ class Attention(Part):
         heads come in pairs per kv head: what the tcgen05 prompt kernel's build with a bias takes."""
         return (self.distance_bias is not None and gate is None and self.sinks is None and not self.softcap
                 and not self.split_weights and (self.n_heads // self.n_kv) % 2 == 0)
+
+    def _slopes_alone(self, gate) -> bool:
+        """Whether the layer's extras are a linear bias by distance and perhaps a sink, with the softmax weights in one
+        bfloat16 term: what the tcgen05 prompt kernel's builds with slopes take."""
+        return (self.distance_slopes is not None and gate is None and self.distance_bias is None and not self.softcap
+                and not self.split_weights)
 
     def _attend_with_extras(self, q, out, table, batch, plan, decode_kernel: bool, prefill_kernel: bool,
                             gate: torch.Tensor | None = None) -> None:
@@ -577,18 +586,23 @@ class Attention(Part):
                                  splits, scratch, batch.status,
                                  extras=ops.attention_extras(q[:n_decode], self.sinks,
                                                              gate[:n_decode] if gate is not None else None,
-                                                             self.split_weights, self.softcap, bias))
+                                                             self.split_weights, self.softcap, bias,
+                                                             self.distance_slopes))
         if n_decode == tokens:
             return
         tiles = plan.get("tiles")
         if prefill_kernel and tiles is not None and n_decode == int(batch.n_decode):
             # (the tile list covers exactly the tokens after the leading single tokens)
-            if self._bias_alone(gate):
-                # A bias by distance and nothing else: the tcgen05 kernel's build that adds it to its products.
+            if self._bias_alone(gate) or self._slopes_alone(gate):
+                # A bias by distance and nothing else (or slopes, and perhaps a sink): the tcgen05 kernel's builds that
+                # add it to their products.
                 if self._prefill_tcgen05 is None:
                     self._prefill_tcgen05 = ops.attention_prefill_tcgen05_supports(q, cache.k_pool, cache.page_size)
                 if self._prefill_tcgen05:
-                    ctas = tiles.shape[0] * (self.n_heads // 2)
+                    odd = (self.n_heads // self.n_kv) % 2 == 1   # (slopes only) a head per CTA, tiles of up to twice the rows
+                    if odd and plan.get("tiles_wide") is not None:
+                        tiles = plan["tiles_wide"]
+                    ctas = tiles.shape[0] * (self.n_heads if odd else self.n_heads // 2)
                     max_keys = int(plan.get("max_keys") or 0)
                     if self.window:
                         max_keys = min(max_keys, self.window + ops.attention_prefill_tile_rows())
@@ -600,17 +614,19 @@ class Attention(Part):
                                               dtype=torch.float32, device=q.device)
                     ops.attention_prefill_tcgen05(q, cache.k_pool, cache.v_pool, table, tiles, out, cache.page_size,
                                                   self.window, self.scale, batch.status, splits, scratch, False,
-                                                  distance_bias=bias)
+                                                  distance_bias=bias, distance_slopes=self.distance_slopes,
+                                                  sinks=self.sinks)
                     return
             ops.attention_prefill(q, cache.k_pool, cache.v_pool, table, tiles, out, cache.page_size, self.window,
                                   self.scale, batch.status,
                                   extras=ops.attention_extras(q, self.sinks, gate, self.split_weights, self.softcap,
-                                                              bias))
+                                                              bias, self.distance_slopes))
             return
         ops.attention_simt(q[n_decode:], cache.k_pool, cache.v_pool, table, batch.pos[n_decode:],
                            batch.entry[n_decode:], out[n_decode:], cache.page_size, self.window, self.scale,
                            batch.status, softcap=self.softcap, sinks=self.sinks,
-                           gate=gate[n_decode:] if gate is not None else None, distance_bias=bias)
+                           gate=gate[n_decode:] if gate is not None else None, distance_bias=bias,
+                           distance_slopes=self.distance_slopes)
 
     def attend(self, q: torch.Tensor, out: torch.Tensor, table: torch.Tensor, batch, rope: tuple | None = None,
                gate: torch.Tensor | None = None) -> None:
@@ -659,7 +675,8 @@ class Attention(Part):
                                    batch.entry[:n_simt], out[:n_simt], cache.page_size, self.window, self.scale,
                                    batch.status, cache.mass_sum, cache.weight_sum, weights[:n_simt],
                                    softcap=self.softcap, sinks=self.sinks,
-                                   gate=gate[:n_simt] if gate is not None else None, distance_bias=self.distance_bias)
+                                   gate=gate[:n_simt] if gate is not None else None, distance_bias=self.distance_bias,
+                                   distance_slopes=self.distance_slopes)
             if fast:
                 ops.attention_prefill_tcgen05(q, cache.k_pool, cache.v_pool, table, tiles, out, cache.page_size,
                                               self.window, self.scale, batch.status, 1, None, wide,

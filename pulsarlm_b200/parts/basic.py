@@ -51,6 +51,30 @@ class ScaledPair:
         return dataclasses.replace(self, also=rows)
 
 
+@dataclasses.dataclass
+class NormedSides:
+    """The outputs of two sublayers side by side that enter the residual stream normed and scaled, beside the plain
+    output of a third that read the same input: x += factor * (rmsnorm(y1 + b1) * w1 + rmsnorm(y2 + b2) * w2) + y3
+    (biases and weights fp32, one eps; b1, b2 and y3 may be None). A block hands it on in the place of a plain
+    delta; the next norm's kernel does the norms, the adds and its own norm in one pass (ops.side_norm)."""
+
+    y1: torch.Tensor
+    b1: torch.Tensor | None
+    w1: torch.Tensor
+    y2: torch.Tensor
+    b2: torch.Tensor | None
+    w2: torch.Tensor
+    factor: float
+    eps: float
+    y3: torch.Tensor | None = None
+
+    def sides(self) -> tuple:
+        return (self.y1, self.b1, self.w1, self.y2, self.b2, self.w2)
+
+    def with_third(self, y: torch.Tensor | None) -> "NormedSides":
+        return dataclasses.replace(self, y3=y)
+
+
 @register_part("norm", "rmsnorm")
 class RMSNorm(Part):
     """h = v * rsqrt(mean(v^2) + eps) * weight over the fp32 residual stream, with
@@ -97,6 +121,10 @@ class RMSNorm(Part):
         elif isinstance(delta, NormedDelta):
             ops.add_normed_rmsnorm(x, delta.y, delta.weight, delta.mult, delta.eps, self.weight_f32(), self.eps, out,
                                    rows, delta.bias, conv)
+        elif isinstance(delta, NormedSides):
+            if conv is not None:
+                raise ValueError("rmsnorm: a filter cannot ride along with two normed sides")
+            ops.side_norm(x, delta.sides(), delta.factor, delta.eps, delta.y3, self.weight_f32(), self.eps, out, rows)
         else:
             ops.add_rmsnorm(x, delta, self.weight, self.eps, out, rows)
         return out
@@ -129,6 +157,8 @@ def settle_pending(x: torch.Tensor, delta) -> None:
     elif isinstance(delta, NormedDelta):
         ops.add_normed_rmsnorm(x, delta.y, delta.weight, delta.mult, delta.eps, delta.weight, delta.eps, None, None,
                                delta.bias)
+    elif isinstance(delta, NormedSides):
+        ops.side_norm(x, delta.sides(), delta.factor, delta.eps, delta.y3, None, 0.0, None)
     elif isinstance(delta, torch.Tensor):
         x.add_(delta)
     else:
@@ -374,8 +404,9 @@ class PairHashEmbedding(Part):
 
 @register_part("head", "linear")
 class Head(Part):
-    """logits = h W^T in fp32, times `scale` where given. params: vocab_size, hidden_size, scale
-    (optional, 1 when absent). tensors: weight
+    """logits = h W^T in fp32, times `scale` where given, then softcap * tanh(logits / softcap)
+    where that is given. params: vocab_size, hidden_size, scale
+    (optional, 1 when absent), softcap (optional). tensors: weight
     [vocab, hidden], or None for a head tied to the embedding table, which the
     model then hands over with `tie`. The reference ties when the weights hold
     no lm_head.weight (pulsarlm-core/src/engine/model/llama.cpp:31); here
@@ -386,6 +417,7 @@ class Head(Part):
         self.vocab = int(self.param("vocab_size"))
         self.hidden = int(self.param("hidden_size"))
         self.scale = float(spec.params.get("scale") or 1.0)
+        self.softcap = float(spec.params.get("softcap") or 0.0)
         self.weight: torch.Tensor | None = None
 
     @property
@@ -414,7 +446,9 @@ class Head(Part):
 
     def forward(self, h: torch.Tensor) -> torch.Tensor:
         logits = linear(h, self.weight, out_dtype=torch.float32)
-        if self.scale != 1.0:
+        if self.softcap:
+            ops.capped_scale(logits, self.scale, self.softcap)
+        elif self.scale != 1.0:
             logits.mul_(self.scale)
         return logits
 
@@ -422,8 +456,10 @@ class Head(Part):
 @register_part("feed_forward", "gated_mlp")
 class GatedMLP(Part):
     """(act(h Wg^T) * (h Wu^T)) Wd^T with act = SiLU
-    (pulsarlm-core/src/engine/model/llama.cpp:91) or the tanh form of GELU. params:
-    hidden_size, intermediate_size, activation ("silu", the default, or "gelu_tanh").
+    (pulsarlm-core/src/engine/model/llama.cpp:91) or the tanh form of GELU, or with the clamped
+    unit in the place of act(g) * u: g cut off above at `limit`, u on both sides, g sigmoid(1.702 g)
+    (u + 1). params: hidden_size, intermediate_size, activation ("silu", the default, "gelu_tanh" or
+    "clamped"), limit ("clamped").
     tensors: gate, up [I, H], down [H, I].
     gate and up are stacked into one [2I, H] operand at load."""
 
@@ -432,9 +468,10 @@ class GatedMLP(Part):
         self.hidden = int(self.param("hidden_size"))
         self.inter = int(self.param("intermediate_size"))
         self.activation = str(spec.params.get("activation") or "silu")
-        if self.activation not in ("silu", "gelu_tanh"):
+        if self.activation not in ("silu", "gelu_tanh", "clamped"):
             raise ValueError(f"gated_mlp: unsupported activation {self.activation!r} (supported: 'silu', "
-                             f"'gelu_tanh')")
+                             f"'gelu_tanh', 'clamped')")
+        self.limit = float(self.param("limit")) if self.activation == "clamped" else 0.0
         self.gate_up: torch.Tensor | None = None
         self.down: torch.Tensor | None = None
 
@@ -450,7 +487,7 @@ class GatedMLP(Part):
         self.down = tensors[t["down"]].contiguous()
 
     def forward(self, h: torch.Tensor, batch) -> torch.Tensor:
-        return gated_feed_forward(h, self.gate_up, self.down, self.activation)
+        return gated_feed_forward(h, self.gate_up, self.down, self.activation, self.limit)
 
 
 @register_part("feed_forward", "mlp")

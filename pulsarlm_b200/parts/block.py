@@ -203,7 +203,10 @@ class ParallelBlock:
         x += scale_mixer * mixer(norm_mixer(x)) + scale_ff * feed_forward(norm_ff(x))
 
     Norm names in the LayerSpec: "mixer" and "feed_forward" (the latter only where the layer
-    has a feed-forward). `extras`: "mixer_scale" / "feed_forward_scale", checkpoint names of
+    has a feed-forward; a layer that has one and names no norm for it feeds it the mixer's normed
+    input). A mixer that hands its output on as something pending of its own (`pending`: outputs that
+    are normed on their way into the stream) takes the feed-forward's along in the place of a
+    ScaledPair; such a layer has no scales. `extras`: "mixer_scale" / "feed_forward_scale", checkpoint names of
     the per-channel scales [hidden] (absent: unscaled). The sum is not formed here: the
     outputs travel as a ScaledPair and the next block's norm kernel scales them, adds them
     into the fp32 stream and writes both of its norms in one pass."""
@@ -216,8 +219,12 @@ class ParallelBlock:
         self.mixer = build_part("mixer", spec.mixer, ctx)
         self.feed_forward = self.ff_norm = None
         if spec.feed_forward is not None:
-            self.ff_norm = build_part("norm", spec.norms["feed_forward"], ctx)
+            if spec.norms.get("feed_forward") is not None:
+                self.ff_norm = build_part("norm", spec.norms["feed_forward"], ctx)
             self.feed_forward = build_part("feed_forward", spec.feed_forward, ctx)
+        self._pending = hasattr(self.mixer, "pending")
+        if self._pending and (extras.get("mixer_scale") or extras.get("feed_forward_scale")):
+            raise ValueError("parallel: a mixer that norms its own output on the way in takes no scales")
         self.scales = _LayerScales(extras.get("mixer_scale"),
                                    extras.get("feed_forward_scale") if spec.feed_forward is not None else None,
                                    int(spec.norms["mixer"].params["hidden_size"]))
@@ -227,7 +234,9 @@ class ParallelBlock:
         extras = spec.extras or {}
         out = [("norm", spec.norms["mixer"]), ("mixer", spec.mixer)]
         if spec.feed_forward is not None:
-            out += [("norm", spec.norms["feed_forward"]), ("feed_forward", spec.feed_forward)]
+            if spec.norms.get("feed_forward") is not None:
+                out.append(("norm", spec.norms["feed_forward"]))
+            out.append(("feed_forward", spec.feed_forward))
         names = {"mixer": extras.get("mixer_scale"),
                  "feed_forward": extras.get("feed_forward_scale") if spec.feed_forward is not None else None}
         out.append(("block", _scales_spec(names, int(spec.norms["mixer"].params["hidden_size"]))))
@@ -258,6 +267,11 @@ class ParallelBlock:
         else:
             h1 = self.mixer_norm.forward(x, delta)
             h2 = self.ff_norm.forward(x, None) if self.ff_norm is not None else None
+        if self.ff_norm is None:
+            h2 = h1
+        if self._pending:
+            sides = self.mixer.pending(h1, batch)
+            return x, sides.with_third(self.feed_forward.forward(h2, batch) if self.feed_forward is not None else None)
         y1 = self.mixer.forward(h1, batch)
         y2 = self.feed_forward.forward(h2, batch) if self.feed_forward is not None else None
         return x, ScaledPair(y1, self.scales.mixer, y2, self.scales.feed_forward)

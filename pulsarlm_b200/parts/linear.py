@@ -120,8 +120,10 @@ def gated_linear(x: torch.Tensor, gate_up: torch.Tensor) -> torch.Tensor:
 GATED_IN = os.environ.get("PULSARLM_B200_GATED_IN", "1") != "0"  # (0: always the SwiGLU kernel, for comparison)
 
 
-def gated_feed_forward(x: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, act: str = "silu") -> torch.Tensor:
-    """(act(x Wg^T) * (x Wu^T)) Wd^T -> [T, H], act "silu" or "gelu_tanh". With silu, for a handful
+def gated_feed_forward(x: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, act: str = "silu",
+                       limit: float = 0.0) -> torch.Tensor:
+    """(act(x Wg^T) * (x Wu^T)) Wd^T -> [T, H], act "silu", "gelu_tanh" or "clamped" (ops.gated_act, with its
+    `limit`). With silu, for a handful
     of tokens in bfloat16 the down projection's skinny kernel forms the gated activation itself as it
     reads the gate/up projection's output (one launch fewer, the [T, I] activation never written);
     else `gated_linear` followed by `linear`. Another activation: the product, the gating kernel with
@@ -130,7 +132,7 @@ def gated_feed_forward(x: torch.Tensor, gate_up: torch.Tensor, down: torch.Tenso
     inter = gate_up.shape[0] // 2
     if act != "silu":
         gated = torch.empty((tokens, inter), dtype=x.dtype, device=x.device)
-        ops.gated_act(linear(x, gate_up), gated, act)
+        ops.gated_act(linear(x, gate_up), gated, act, limit)
         return linear(gated, down)
     if (GATED_IN and x.dtype == torch.bfloat16 == gate_up.dtype == down.dtype
             and tokens <= ops.GEMM_GATED_IN_MAX_TOKENS and down.stride(1) == 1

@@ -40,8 +40,15 @@ class RoutedExperts(Part):
     True); `expert` = "relu2" makes every expert, and the shared one, W_down relu(W_up h)^2 without
     a gate (default "gated_silu"; such experts have no `expert_gate` / `shared_gate` tensors).
 
+    `expert` = "clamped" gives experts the clamped unit in the place of silu(gate) * up (ops.gated_act) with
+    `expert_limit`, and the shared expert `shared_limit`; `weigh_input` = True puts an expert's weight on its input
+    instead of its output (on the gate and up products, which a linear map makes the same thing); the tensor
+    `shared_gate_row` [1, H], where given, makes the shared expert join times sigmoid of its product with h (fp32,
+    a row more in the router's kernel).
+
     params: hidden_size, expert_size, n_experts, top, groups (default 1), keep_groups
-    (default groups), shared_size (optional), scores, group_top, renormalise, expert. tensors: router [E, H], correction [E]
+    (default groups), shared_size (optional), scores, group_top, renormalise, expert, expert_limit, shared_limit,
+    weigh_input. tensors: router [E, H], correction [E]
     (optional), experts: a name pattern with `{e}` for gate / up / down
     (`expert_gate`, `expert_up` [F, H], `expert_down` [H, F]), shared_gate, shared_up [Fs, H],
     shared_down [H, Fs]."""
@@ -59,7 +66,14 @@ class RoutedExperts(Part):
         self.sigmoid_scores = {"softmax": False, "sigmoid": True}[str(p.get("scores") or "softmax")]
         self.group_top = int(p.get("group_top") or 1)
         self.renormalise = bool(p.get("renormalise", True))
-        self.gated = {"gated_silu": True, "relu2": False}[str(p.get("expert") or "gated_silu")]
+        expert = str(p.get("expert") or "gated_silu")
+        self.gated = {"gated_silu": True, "relu2": False, "clamped": True}[expert]
+        self.limit = float(self.param("expert_limit")) if expert == "clamped" else None
+        self.shared_limit = float(self.param("shared_limit")) if expert == "clamped" and self.shared_size else None
+        self.weigh_input = bool(p.get("weigh_input", False))
+        if self.weigh_input and self.limit is None:
+            raise ValueError("moe: only experts with the clamped unit take their weight on the input")
+        self.shared_gate_row = bool(spec.tensors.get("shared_gate_row")) and self.shared_size > 0
         if self.n_experts % self.groups or not 0 < self.keep <= self.groups:
             raise ValueError(f"moe: {self.n_experts} experts in {self.groups} groups of which {self.keep} stay")
         if not 0 < self.top <= self.keep * (self.n_experts // self.groups):
@@ -74,7 +88,7 @@ class RoutedExperts(Part):
     def tensor_needs(cls, spec: PartSpec) -> dict[str, TensorNeed]:
         p, t = spec.params, spec.tensors
         h, f, e = int(p["hidden_size"]), int(p["expert_size"]), int(p["n_experts"])
-        gated = str(p.get("expert") or "gated_silu") == "gated_silu"
+        gated = str(p.get("expert") or "gated_silu") in ("gated_silu", "clamped")
         needs = {t["router"]: TensorNeed((e, h))}
         if t.get("correction"):
             needs[t["correction"]] = TensorNeed((e,), role="offset")
@@ -89,11 +103,15 @@ class RoutedExperts(Part):
                 needs[t["shared_gate"]] = TensorNeed((fs, h))
             needs[t["shared_up"]] = TensorNeed((fs, h))
             needs[t["shared_down"]] = TensorNeed((h, fs))
+            if t.get("shared_gate_row"):
+                needs[t["shared_gate_row"]] = TensorNeed((1, h))
         return needs
 
     def load(self, tensors: dict[str, torch.Tensor]) -> None:
         t = self.spec.tensors
         self.router = tensors[t["router"]].float().contiguous()
+        if self.shared_gate_row:
+            self.router = torch.cat([self.router, tensors[t["shared_gate_row"]].float()], dim=0).contiguous()
         self.correction = tensors[t["correction"]].float().contiguous() if t.get("correction") else None
         experts = range(self.n_experts)
         if self.gated:
@@ -114,11 +132,14 @@ class RoutedExperts(Part):
 
     def forward(self, h: torch.Tensor, batch) -> torch.Tensor:
         tokens = h.shape[0]
+        shared_weights = torch.empty(tokens, dtype=torch.float32, device=h.device) if self.shared_gate_row else None
         ids, weights = ops.moe_route(h, self.router, self.correction, self.top, self.groups, self.keep,
-                                     self.sigmoid_scores, self.group_top, self.renormalise)
+                                     self.sigmoid_scores, self.group_top, self.renormalise, shared_weights)
+        in_weights, out_weights = (weights, None) if self.weigh_input else (None, weights)
         shared = None
         if self.shared_size and self.gated:
-            shared = gated_feed_forward(h, self.shared_gate_up, self.shared_down)
+            act = "silu" if self.shared_limit is None else "clamped"
+            shared = gated_feed_forward(h, self.shared_gate_up, self.shared_down, act, self.shared_limit or 0.0)
         elif self.shared_size:
             shared = activated_linear(linear(h, self.shared_gate_up), None, "relu2", self.shared_down)
         out = torch.empty((tokens, self.hidden), dtype=h.dtype, device=h.device)
@@ -129,17 +150,19 @@ class RoutedExperts(Part):
             x = ops.moe_gather(h, pair_of_row, self.top)
             gate_up = torch.nn.functional.grouped_mm(x, self.gate_up.transpose(1, 2), offs=ends)
             act = torch.empty((x.shape[0], self.ff), dtype=h.dtype, device=h.device)
-            if self.gated:
+            if self.limit is not None:
+                ops.gated_act(gate_up, act, "clamped", self.limit, in_weights, pair_of_row)
+            elif self.gated:
                 ops.swiglu(gate_up, act)
             else:
                 ops.bias_act(gate_up, None, act, "relu2")
             y = torch.nn.functional.grouped_mm(act, self.down.transpose(1, 2), offs=ends)
-            ops.moe_combine(y, row_of_pair, weights, shared, out)
+            ops.moe_combine(y, row_of_pair, out_weights, shared, out, shared_weights)
             return out
         act = torch.empty((tokens * self.top, self.ff), dtype=h.dtype, device=h.device)
         if self.gated:
-            ops.moe_gate_up(h, self.gate_up, ids, act)
+            ops.moe_gate_up(h, self.gate_up, ids, act, self.limit, in_weights)
         else:
             ops.moe_up(h, self.gate_up, ids, act)
-        ops.moe_down(act, self.down, ids, weights, shared, out)
+        ops.moe_down(act, self.down, ids, out_weights, shared, out, shared_weights)
         return out

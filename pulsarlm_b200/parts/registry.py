@@ -25,6 +25,8 @@ Interfaces (duck-typed; the base classes below document them):
 * filter:      something a block puts in front of a sublayer's input (a short convolution
                over time): `forward(h, batch) -> [T, H]` engine dtype, and like a mixer
                `cache_need()` / `bind_cache(binding)` when it keeps state per request.
+* join:        what replaces the stream before a pass of repeated layers: `forward(x, delta, entered)
+               -> x` with the stream, what is pending and the stream as it entered the first layer.
 * block:       `forward(x, delta, batch) -> (x, delta)`: the arrangement of
                norms, mixer and feed-forward around the residual stream.
 """
@@ -38,7 +40,7 @@ import torch
 
 from .spec import PartSpec, TensorNeed
 
-_KINDS = ("norm", "position", "mixer", "feed_forward", "block", "embedding", "head", "filter")
+_KINDS = ("norm", "position", "mixer", "feed_forward", "block", "embedding", "head", "filter", "join")
 _REGISTRIES: dict[str, dict[str, type]] = {k: {} for k in _KINDS}
 
 
@@ -72,8 +74,9 @@ def _load_builtins() -> None:
     global _builtins_loaded
     if not _builtins_loaded:
         _builtins_loaded = True
-        from . import (attention, basic, block, conv_attention, delta_rule, diff_attention, gated_delta,  # noqa: F401
-                       latent_attention, moe, normed_attention, short_conv)
+        from . import (attention, basic, block, conv_attention, delta_rule, diff_attention,  # noqa: F401
+                       filtered_attention, gated_delta, latent_attention, linear_recurrence, moe, normed_attention,
+                       short_conv, side_by_side, stream_join)
 
 
 def part_class(kind: str, name: str) -> type:

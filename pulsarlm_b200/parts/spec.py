@@ -46,7 +46,9 @@ class ModelSpec:
     cache or state of its own (a layer that runs twice then has two, one per run),
     and the cache manager is asked run by run instead of layer by layer.
     `rejoin_runs`: places in `order` before which the embedding's output (the
-    stream as it entered the first layer) is added to the stream again."""
+    stream as it entered the first layer) is added to the stream again. `join` with
+    `join_runs`: a part of the "join" registry that makes a new stream of the stream and
+    the embedding's output before those places in `order` (the first place too, if listed)."""
 
     hidden_size: int
     vocab_size: int
@@ -59,6 +61,8 @@ class ModelSpec:
     max_position_embeddings: int | None = None
     cache_per_run: bool = False
     rejoin_runs: tuple[int, ...] = ()
+    join: PartSpec | None = None
+    join_runs: tuple[int, ...] = ()
 
 
 @dataclasses.dataclass(frozen=True)
