@@ -84,7 +84,7 @@ __global__ void __launch_bounds__(kThreads) conv_qkv_write_kernel(const ConvQkvP
     }
     pl_grid_wait();
     const int t0 = blockIdx.x * p.tokens_per_block, t1 = min(t0 + p.tokens_per_block, p.n_tokens);
-    typename Piece::Raw window[kReach];  // (TAPS > 0) the inputs before the token at hand, oldest first
+    float window[kReach][PER];  // (TAPS > 0) the inputs before the token at hand, oldest first, with the bias
     int last_entry = -1;
     for (int t = t0; t < t1; ++t) {
         const int e = p.entry[t], at = p.pos[t];
@@ -110,38 +110,40 @@ __global__ void __launch_bounds__(kThreads) conv_qkv_write_kernel(const ConvQkvP
             float v[PER];
             if constexpr (TAPS > 0) {
                 if (fresh) {
+                    typename Piece::Raw raw[kReach];
 #pragma unroll
                     for (int j = 0; j < TAPS - 1; ++j) {
-                        window[j] = earlier(TAPS - 1 - j);
+                        raw[j] = earlier(TAPS - 1 - j);
                     }
-                }
 #pragma unroll
-                for (int j = 0; j < TAPS - 1; ++j) {
-                    if (at - (TAPS - 1 - j) >= 0) {
-                        Piece::floats(window[j], v);
+                    for (int j = 0; j < TAPS - 1; ++j) {
+                        Piece::floats(raw[j], v);
 #pragma unroll
                         for (int i = 0; i < PER; ++i) {
-                            y[i] = fmaf(w[j][i], v[i] + b[i], y[i]);
+                            window[j][i] = at - (TAPS - 1 - j) >= 0 ? v[i] + b[i] : 0.0f;
+                        }
+                    }
+                    if (p.update_state) {
+#pragma unroll
+                        for (int j = 0; j < TAPS - 1; ++j) {
+                            Piece::put(old + static_cast<int64_t>(j) * p.channels, j + 1 < TAPS - 1 ? raw[j + 1] : own);
                         }
                     }
                 }
                 Piece::floats(own, v);
 #pragma unroll
                 for (int i = 0; i < PER; ++i) {
-                    y[i] = fmaf(w[TAPS - 1][i], v[i] + b[i], y[i]);
-                }
-#pragma unroll
-                for (int j = 0; j + 1 < TAPS - 1; ++j) {
-                    window[j] = window[j + 1];
-                }
-                if (TAPS > 1) {
-                    window[kReach - 1] = own;
-                }
-                if (p.update_state) {
+                    v[i] += b[i];
 #pragma unroll
                     for (int j = 0; j < TAPS - 1; ++j) {
-                        Piece::put(old + static_cast<int64_t>(j) * p.channels, window[j]);
+                        y[i] = fmaf(w[j][i], window[j][i], y[i]);
                     }
+                    y[i] = fmaf(w[TAPS - 1][i], v[i], y[i]);
+#pragma unroll
+                    for (int j = 0; j + 1 < TAPS - 1; ++j) {
+                        window[j][i] = window[j + 1][i];
+                    }
+                    window[kReach - 1][i] = v[i];
                 }
             } else {
                 for (int j = 0; j < taps; ++j) {
