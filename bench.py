@@ -1135,6 +1135,195 @@ def puvirax_kernels(width: int, pk: dict) -> dict:
     return out
 
 
+def pakarax_config(width: int, runs: int, vocab: int = 32000) -> dict:
+    """A Pakarax model at a real model's layer sizes with `runs` layer runs: heads of 64 in groups of four, four taps on
+    either side, a recurrence as wide as the model in gate blocks of 256; a dense feed-forward of 8/3 x width alternating
+    with 16 routed experts of 2/3 x width (2 chosen) beside a shared expert of 4/3 x width (the same active size). The
+    middle layers run twice, each pass entered through the projection that joins the stream with the embedding."""
+    heads, kv = width // 64, max(1, width // 256)
+    ff = (8 * width // 3 + 255) // 256 * 256
+    dense = {"kind": "dense", "ff": ff, "limit": 7.0}
+    routed = {"kind": "moe", "expert": {"ff": ff // 4, "limit": 7.0}, "shared": {"ff": ff // 2, "limit": 7.0},
+              "router": {"experts": 16, "top": 2}}
+    mixer = {"left": {"heads": heads, "kv_heads": kv, "dim": 64, "vdim": 64, "conv": 4, "scale": 0.125,
+                      "q_temp": {"coef": 0.1, "every": 1024}},
+             "right": {"width": width, "blocks": width // 256, "conv": 4}}
+    looped = [routed, dense] if runs % 2 == 0 else [routed]
+    mlps = [dense] + looped + [routed] * (runs - 1 - 2 * len(looped))
+    return {"architecture": "Pakarax", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "logit_scale": 0.5,
+            "logit_softcap": 30.0, "loop": {"start": 1, "stop": 1 + len(looped), "times": 2},
+            "layers": [{"type": "parallel", "mixer": mixer, "mlp": mlp} for mlp in mlps]}
+
+
+def pakarax_kernels(width: int, pk: dict) -> dict:
+    """The Pakarax design's kernels alone at one layer's sizes, each beside the like kernel of the Llama layer (or of the
+    design named): milliseconds, algorithmic bytes or FLOPs, fraction of the copy bandwidth."""
+    import torch
+
+    from pulsarlm_b200.kernels import ops
+    from pulsarlm_b200.parts.filtered_attention import geometric_slopes
+
+    dev, bf = "cuda:0", torch.bfloat16
+    out: dict = {}
+
+    def note(name, ms, nbytes=None, flops=None):
+        out[name] = {"ms": ms}
+        if nbytes is not None:
+            out[name].update(bytes=nbytes, frac_of_hbm=nbytes / (ms / 1e3) / 1e9 / pk["hbm_gbs"])
+        if flops is not None:
+            out[name].update(tflops=flops / (ms / 1e3) / 1e12, frac_of_bf16=flops / (ms / 1e3) / 1e12 / pk["bf16_tflops"])
+
+    def f32(*shape):
+        return torch.randn(shape, device=dev)
+
+    def b16(*shape):
+        return f32(*shape).to(bf)
+
+    heads, kv, hd, page, taps, block = width // 64, max(1, width // 256), 64, 16, 4, 256
+    blocks = width // block
+    experts, top, ff = 16, 2, (8 * width // 3 + 255) // 256 * 64
+    channels = (heads + 2 * kv) * hd
+    bias, conv = f32(channels), f32(taps, channels)
+    x_bias, y_bias, conv_bias, ra_bias, ri_bias = (f32(width) for _ in range(5))
+    ring_conv_w, decay, gates = f32(taps, width), -torch.rand(width, device=dev), b16(blocks, 2 * block, block)
+    router, router_shared = f32(experts, width), f32(experts + 1, width)
+    gate_up, down = b16(experts, 2 * ff, width), b16(experts, width, ff)
+    w1, w2, w3 = f32(width), f32(width), f32(width)
+    for tokens, entries in ((2048, 1), (8, 8), (64, 64)):
+        tag = f"T{tokens}_E{entries}"
+        per = tokens // entries
+        entry = torch.arange(entries, dtype=torch.int32, device=dev).repeat_interleave(per)
+        slots = torch.arange(entries, dtype=torch.int32, device=dev)
+        first = torch.arange(0, tokens, per, dtype=torch.int32, device=dev)
+        count = torch.full((entries,), per, dtype=torch.int32, device=dev)
+        pos = torch.arange(8, per + 8, dtype=torch.int32, device=dev).repeat(entries)
+        n_pages = entries * ((per + 8) // page + 1)
+        table = torch.arange(n_pages, dtype=torch.int32, device=dev).view(entries, -1)
+        # projection -> convolution, temperature, cache write
+        proj = b16(tokens, channels + 2 * width)
+        stride = channels + 2 * width
+        pools = torch.zeros((2, n_pages, kv, page, hd), dtype=bf, device=dev)
+        q_out = torch.empty((tokens, heads, hd), dtype=bf, device=dev)
+        state = torch.zeros((entries, taps - 1, channels), dtype=bf, device=dev)
+        note(f"conv_qkv_write_{tag}",
+             time_kernel(lambda: ops.conv_qkv_write(proj[:, :channels], stride, bias, conv, state, slots, per == 1, 0.1, 1024,
+                                                    pos, entry, table, q_out, pools[0], pools[1], page, kv, hd, hd, heads * hd,
+                                                    (heads + kv) * hd)),
+             tokens * channels * 2 * 2 + (2 * entries * (taps - 1) * channels * 2 if per == 1 else 0))
+        filtered = torch.empty((tokens, channels), dtype=bf, device=dev)
+        wide_conv = conv.t().contiguous()
+        if per > 1:
+            note(f"short_conv_silu_{tag} (Bunosun, the same channels)",
+                 time_kernel(lambda: ops.short_conv_act(proj[:, :channels], wide_conv, state, entry, slots, filtered,
+                                                        residual=False, act="silu")), tokens * channels * 2 * 2)
+        inv = torch.rand(hd // 2, dtype=torch.float64, device=dev)
+        q, k, v = (proj[:, :heads * hd].view(tokens, heads, hd),
+                   proj[:, heads * hd:(heads + kv) * hd].view(tokens, kv, hd),
+                   proj[:, (heads + kv) * hd:channels].view(tokens, kv, hd))
+        note(f"rope_kv_write_{tag} (Llama)",
+             time_kernel(lambda: ops.rope_kv_write(q, k, v, pos, entry, table, pools[0], pools[1], page, inv, hd, None)),
+             tokens * (heads * hd * 2 * 2 + kv * hd * 2 * 4))
+        # the recurrence
+        x, y = proj[:, channels:channels + width], proj[:, channels + width:]
+        ring = torch.zeros((entries, taps, width), dtype=bf, device=dev)
+        states = torch.zeros((entries, width), device=dev)
+        res = torch.empty((tokens, width), dtype=bf, device=dev)
+        if per > 1:
+            u = torch.empty((tokens, width), dtype=bf, device=dev)
+            note(f"ring_conv_{tag}", time_kernel(lambda: ops.ring_conv(x, stride, x_bias, ring_conv_w, conv_bias, ring, first,
+                                                                       entry, slots, pos, u)), tokens * width * 4)
+
+            def products():
+                return torch.bmm(u.view(tokens, blocks, block).transpose(0, 1), gates.transpose(1, 2), out_dtype=torch.float32)
+
+            pre = products()
+            note(f"gate_products_{tag} (library)", time_kernel(products), tokens * width * (2 + 8),
+                 4.0 * tokens * width * block)
+            note(f"linear_scan_{tag}",
+                 time_kernel(lambda: ops.linear_scan(pre, ra_bias, ri_bias, decay, u, y, y_bias, x, stride, ring, states,
+                                                     first, count, slots, pos, per, res)), tokens * width * (8 + 2 + 2 + 2))
+        else:
+            note(f"linear_step_{tag}",
+                 time_kernel(lambda: ops.linear_step(x, stride, x_bias, ring_conv_w, conv_bias, ring, gates, ra_bias, ri_bias,
+                                                     decay, y, y_bias, states, entry, slots, pos, res)),
+                 gates.numel() * 2 + tokens * width * (2 * 2 + 2 * taps + 8 + 2))
+        nh = width // 64
+        qk = b16(tokens, 3 * nh * 64)
+        delta_states = torch.zeros((entries, nh, 64, 64), device=dev)
+        a_log, dt, norm = f32(nh), f32(nh * 64), torch.ones(64, device=dev)
+        b_pre, a_pre, g_pre = b16(tokens, nh), b16(tokens, nh * 64), b16(tokens, nh * 64)
+        note(f"gated_delta_{tag} (Bunosun)",
+             time_kernel(lambda: ops.gated_delta(qk[:, :nh * 64], qk[:, nh * 64:2 * nh * 64], qk[:, 2 * nh * 64:], b_pre, a_pre,
+                                                 g_pre, a_log, dt, norm, delta_states, first, count, slots, res, nh, nh, 64, 64,
+                                                 1e-6, 0.125, 1e-6)),
+             tokens * width * 12 + 2 * delta_states.numel() * 4)
+        # the residual add and the norms
+        stream, y1, y2, y3 = f32(tokens, width), b16(tokens, width), b16(tokens, width), b16(tokens, width)
+        h = torch.empty((tokens, width), dtype=bf, device=dev)
+        note(f"side_norm_{tag}", time_kernel(lambda: ops.side_norm(stream, (y1, w1, w2, y2, None, w3), 0.5, 1e-6, y3, w1, 1e-6,
+                                                                   h)), tokens * width * (8 + 6 + 2))
+        note(f"add_rmsnorm_{tag} (Llama)", time_kernel(lambda: ops.add_rmsnorm(stream, y1, w1, 1e-6, h)),
+             tokens * width * (8 + 2 + 2))
+        both = torch.empty((tokens, 2 * width), dtype=bf, device=dev)
+        note(f"side_norm_join_{tag}", time_kernel(lambda: ops.side_norm(stream, (y1, w1, w2, y2, None, w3), 0.5, 1e-6, y3, None,
+                                                                        0.0, both, entered=stream)),
+             tokens * width * (8 + 6 + 4 + 4))
+        # the feed-forward's unit, the router, the experts pair by pair
+        z = b16(tokens, 8 * ff)
+        unit = torch.empty((tokens, 4 * ff), dtype=bf, device=dev)
+        note(f"gated_act_clamped_{tag}", time_kernel(lambda: ops.gated_act(z, unit, "clamped", 7.0)), tokens * 4 * ff * 6)
+        note(f"swiglu_{tag} (Llama)", time_kernel(lambda: ops.swiglu(z, unit)), tokens * 4 * ff * 6)
+        shared = torch.empty(tokens, device=dev)
+        route_bytes = tokens * width * 2 + experts * width * 4
+        note(f"moe_route_sigmoid_shared_{tag}",
+             time_kernel(lambda: ops.moe_route(h, router_shared, None, top, 1, 1, True, 1, False, shared)), route_bytes)
+        note(f"moe_route_softmax_{tag} (Bunosun)", time_kernel(lambda: ops.moe_route(h, router, None, top, 1, 1)), route_bytes)
+        if tokens <= 8:
+            ids, weights = ops.moe_route(h, router, None, top, 1, 1, True, 1, False)
+            act = torch.empty((tokens * top, ff), dtype=bf, device=dev)
+            used = int(ids.unique().numel())
+            note(f"moe_gate_up_clamped_{tag}", time_kernel(lambda: ops.moe_gate_up(h, gate_up, ids, act, 7.0, weights)),
+                 used * 2 * ff * width * 2)
+            note(f"moe_gate_up_{tag} (Bunosun)", time_kernel(lambda: ops.moe_gate_up(h, gate_up, ids, act)),
+                 used * 2 * ff * width * 2)
+            note(f"moe_down_shared_gate_{tag}", time_kernel(lambda: ops.moe_down(act, down, ids, None, y1, res, shared)),
+                 used * ff * width * 2)
+            note(f"moe_down_{tag} (Bunosun)", time_kernel(lambda: ops.moe_down(act, down, ids, weights, y1, res)),
+                 used * ff * width * 2)
+    # attention: slopes and sinks beside the Llama layer's kernels
+    sinks, slopes = f32(heads), torch.tensor(geometric_slopes(heads, 8.0), device=dev)
+    keys, batch = 2048, 64
+    n_pages = batch * keys // page
+    table = torch.arange(n_pages, dtype=torch.int32, device=dev).view(batch, keys // page)
+    pos = torch.full((batch,), keys - 1, dtype=torch.int32, device=dev)
+    ent = torch.arange(batch, dtype=torch.int32, device=dev)
+    q, kvp = b16(batch, heads, hd), b16(2, n_pages, kv, page, hd)
+    res = torch.empty_like(q)
+    for splits in (1, 4):
+        scratch = torch.empty(ops.attention_decode_scratch_floats(batch, heads, hd, splits), device=dev)
+        for what, ex in (("slopes_sink", ops.attention_extras(q, sinks, None, False, 0.0, None, slopes)), ("(Llama)", None)):
+            note(f"attention_decode_b64_splits{splits} {what}",
+                 time_kernel(lambda: ops.attention_decode(q, kvp[0], kvp[1], table, pos, ent, res, page, None, 0.125, splits,
+                                                          scratch, extras=ex)), batch * keys * kv * hd * 4)
+    tokens = 2048
+    n_pages = tokens // page
+    table = torch.arange(n_pages, dtype=torch.int32, device=dev).view(1, n_pages)
+    rows = ops.attention_prefill_tile_rows()
+    tiles = torch.tensor([(r, min(rows, tokens - r), r, 0) for r in range(tokens - rows, -1, -rows)], dtype=torch.int32, device=dev)
+    flops = 4.0 * width * tokens * (tokens + 1) / 2
+    for dim in (64, 128):
+        nh, nkv = width // dim, max(1, width // dim // 4)
+        q, kvp = b16(tokens, nh, dim), b16(n_pages, 2, nkv, page, dim)
+        res = torch.empty_like(q)
+        for what, sl, sk in (("slopes, sink", torch.tensor(geometric_slopes(nh, 8.0), device=dev), f32(nh)), ("Llama", None, None)):
+            note(f"attention_prefill_tcgen05_T2048_d{dim} ({what})",
+                 time_kernel(lambda: ops.attention_prefill_tcgen05(q, kvp[:, 0], kvp[:, 1], table, tiles, res, page, None, 0.125,
+                                                                   distance_slopes=sl, sinks=sk)), None, flops)
+    logits = f32(64, 32000)
+    note("capped_scale_R64_V32000", time_kernel(lambda: ops.capped_scale(logits, 0.5, 30.0)), logits.numel() * 8)
+    return out
+
+
 def run_design(args) -> dict:
     """Prefill and decode throughput of the named design at a few sizes beside the Llama
     decoder at the same width, depth and vocabulary (random weights), and the design's own
@@ -1152,7 +1341,7 @@ def run_design(args) -> dict:
     with ClockSampler() as clocks:
         for width, layers in ((1024, 6), (2048, 6), (4096, 3)):
             mine = {"bunosun": bunosun_config, "rerilorn": rerilorn_config, "simetar": simetar_config,
-                    "puvirax": puvirax_config}[args.design](width, layers)
+                    "puvirax": puvirax_config, "pakarax": pakarax_config}[args.design](width, layers)
             for name, cfg in ((args.design, mine), ("llama", llama_config_like(width, layers))):
                 vocab = cfg.get("vocab", cfg.get("vocab_size"))
                 n_pages = (batch * (context + 256) + 4 * prompt) // PAGE_SIZE
@@ -1176,6 +1365,10 @@ def run_design(args) -> dict:
                 decode_ms, launches = time_decode(engine, ids, args.steps, args.warmup, vocab)
                 params = sum(int(t.numel()) for part in engine.model.parts() for t in vars(part).values()
                              if isinstance(t, torch.Tensor))
+                for inner in (i for part in engine.model.parts() for i in getattr(part, "inner_parts", lambda: [])()):
+                    # (parts inside others; their projections of a shared input are rows of an operand counted above)
+                    params += sum(int(t.numel()) for n, t in vars(inner).items()
+                                  if isinstance(t, torch.Tensor) and n not in ("in_weight", "states"))
                 results[f"{name}_w{width}_l{layers}"] = {
                     "parameters": params, "prefill_ms": prefill_ms, "prefill_tok_s": prompt / (prefill_ms / 1e3),
                     "decode_ms": decode_ms, "decode_tok_s": batch / (decode_ms / 1e3),
@@ -1185,7 +1378,7 @@ def run_design(args) -> dict:
                 gc.collect()
                 torch.cuda.empty_cache()
         kernels = {"bunosun": bunosun_kernels, "rerilorn": design_kernels, "simetar": simetar_kernels,
-                   "puvirax": puvirax_kernels}[args.design](2048, pk)
+                   "puvirax": puvirax_kernels, "pakarax": pakarax_kernels}[args.design](2048, pk)
     summary = clocks.summary()
     return {"metric": f"prefill and decode tok/s of the {args.design.capitalize()} design beside the Llama decoder at "
                       f"equal sizes",
@@ -1199,9 +1392,9 @@ def run_design(args) -> dict:
 
 def main() -> int:
     p = argparse.ArgumentParser()
-    p.add_argument("--design", default="llama", choices=["llama", "rerilorn", "bunosun", "simetar", "puvirax"],
-                   help="llama: the headline workload (the default); rerilorn, bunosun, simetar, puvirax: that design's prefill and "
-                        "decode throughput at a few sizes beside the Llama decoder at equal sizes, and its kernels alone")
+    p.add_argument("--design", default="llama", choices=["llama", "rerilorn", "bunosun", "simetar", "puvirax", "pakarax"],
+                   help="llama: the headline workload (the default); rerilorn, bunosun, simetar, puvirax, pakarax: that design's "
+                        "prefill and decode throughput at a few sizes beside the Llama decoder at equal sizes, and its kernels alone")
     p.add_argument("--gpus", type=int, default=1)
     p.add_argument("--steps", type=int, default=128)
     p.add_argument("--warmup", type=int, default=8)
@@ -1223,7 +1416,7 @@ def main() -> int:
         print(f"bench.py measures a single-GPU engine: --gpus {args.gpus} is not supported, run with --gpus 1")
         return 2
     args.warmup = max(3, args.warmup)
-    if args.design in ("rerilorn", "bunosun", "simetar", "puvirax"):
+    if args.design in ("rerilorn", "bunosun", "simetar", "puvirax", "pakarax"):
         args.steps = min(args.steps, 64)
         print(json.dumps(run_design(args)))
         return 0
