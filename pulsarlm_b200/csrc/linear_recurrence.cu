@@ -12,7 +12,7 @@
 // token's inputs need not agree on when the ring moves on.
 //
 // Steps with prompt portions run three kernels: ring_conv (u), the block-diagonal products (elsewhere: [blocks, T,
-// 2 * block] in fp32), and scan, which walks each portion in order. Steps of single tokens in bfloat16 run `step`,
+// 2 * block] in fp32), and the scan over each portion. Steps of single tokens in bfloat16 run `step`,
 // one launch for all of it. Gates, decays, the state and its products are fp32.
 #include "cluster_helpers.cuh"
 #include "row_piece.cuh"
@@ -102,54 +102,94 @@ __global__ void __launch_bounds__(128) ring_conv_kernel(
 }
 
 // ------------------------------------------------------------------------------------------------ scan
-// A cluster of CTAs takes 64 channels of one entry's portion, each CTA the next kSpan tokens in turn: all threads form
-// (a, b) of the CTA's tokens in shared memory at once; then the CTAs walk their tokens one after the other, a thread
-// per channel, and hand the state on through distributed shared memory; then all threads multiply by the other
-// branch and store. The walk is the plain recurrence in token order, whatever the cluster's size.
+// A cluster of CTAs takes 64 channels of one entry's portion, each CTA the next kSpan tokens in turn. Two forms:
+//
+// * walked (float32): all threads form (a, b) of the CTA's tokens in shared memory at once; then the CTAs walk their
+//   tokens one after the other, a thread per channel, and hand the state on through distributed shared memory; then
+//   all threads multiply by the other branch and store. The walk is the plain recurrence in token order, whatever the
+//   cluster's size: a portion's cut changes no bit.
+// * composed (bfloat16): a thread takes kSub neighbouring tokens of a channel, (a, b) and the other branch in
+//   registers, and composes them into one step S -> A S + B; a CTA's threads' steps compose into the CTA's, which goes to
+//   every CTA's shared memory. One barrier of the cluster makes the steps visible, every thread folds those before its
+//   own into its start, and walks its tokens from there. The fp32 sums differ from the walked form's in their last
+//   bits only.
 constexpr int kChannels = 64;
 constexpr int kSpan = 128;
 constexpr int kScanThreads = 256;
 constexpr int kScanShared = 2 * kSpan * kChannels * static_cast<int>(sizeof(float));
+constexpr int kSubs = kScanThreads / kChannels;
+constexpr int kSub = kSpan / kSubs;
+constexpr int kMaxCluster = 8;
 
 __device__ __forceinline__ void cluster_store1(uint32_t remote, float v) {
     asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(remote), "f"(v) : "memory");
 }
+__device__ __forceinline__ void cluster_store2(uint32_t remote, float2 v) {
+    asm volatile("st.shared::cluster.v2.f32 [%0], {%1, %2};" ::"r"(remote), "f"(v.x), "f"(v.y) : "memory");
+}
 
+struct ScanParams {
+    const float* pre;  // [blocks, T, 2 * block]
+    const float* ra_bias;
+    const float* ri_bias;
+    const float* decay;
+    const void* u;  // [T, width]
+    const void* y;
+    int64_t y_stride;
+    const float* y_bias;
+    const void* x;
+    int64_t x_stride;
+    void* ring;  // [slots, taps, width]
+    int taps;
+    float* states;  // [slots, width]
+    const int32_t* first;
+    const int32_t* count;
+    const int32_t* slots;
+    const int32_t* pos;
+    void* out;  // [T, width]
+    int n_tokens, width, block, cluster;
+};
+
+// The ring after an entry's portion (the convolution's kernel, which read it, has finished).
 template <typename scalar_t>
-__global__ void __launch_bounds__(kScanThreads) linear_scan_kernel(
-        const float* __restrict__ pre, const float* __restrict__ ra_bias, const float* __restrict__ ri_bias,
-        const float* __restrict__ decay, const scalar_t* __restrict__ u, const scalar_t* __restrict__ y, int64_t y_stride,
-        const float* __restrict__ y_bias, const scalar_t* __restrict__ x, int64_t x_stride, scalar_t* __restrict__ ring,
-        int taps, float* __restrict__ states, const int32_t* __restrict__ first, const int32_t* __restrict__ count,
-        const int32_t* __restrict__ slots, const int32_t* __restrict__ pos, scalar_t* __restrict__ out, int n_tokens,
-        int width, int block, int cluster) {
-    constexpr bool kExact = sizeof(scalar_t) == 4;
+__device__ __forceinline__ void move_ring_on(const ScanParams& p, int c, int64_t slot, int64_t start, int n_all, int j0, int step) {
+    const scalar_t* x = static_cast<const scalar_t*>(p.x);
+    scalar_t* ring = static_cast<scalar_t*>(p.ring);
+    for (int j = j0; j < min(p.taps - 1, n_all); j += step) {
+        const int64_t t = start + n_all - 1 - j;
+        ring[(slot * p.taps + p.pos[t] % p.taps) * p.width + c] = x[t * p.x_stride + c];
+    }
+}
+
+__global__ void __launch_bounds__(kScanThreads) linear_scan_walked_kernel(const ScanParams p) {
     extern __shared__ __align__(16) float terms[];  // [kSpan][kChannels] a, then the same of b (then S)
     float* a_s = terms;
     float* b_s = terms + kSpan * kChannels;
     __shared__ float carry[kChannels];
     pl_grid_trigger();
-    const int rank = blockIdx.x % cluster;
+    const int cluster = p.cluster, rank = blockIdx.x % cluster;
     const int lane = threadIdx.x % kChannels, row0 = threadIdx.x / kChannels;
-    constexpr int kRowsAtOnce = kScanThreads / kChannels;
     const int c = (blockIdx.x / cluster) * kChannels + lane;
-    const bool live = c < width;
+    const bool live = c < p.width;
+    const float* u = static_cast<const float*>(p.u);
+    const float* y = static_cast<const float*>(p.y);
+    float* out = static_cast<float*>(p.out);
     float rb = 0.0f, ib = 0.0f, dc = 0.0f, yb = 0.0f;
     if (live) {
-        rb = ra_bias[c];
-        ib = ri_bias[c];
-        dc = decay[c];
-        yb = y_bias[c];
+        rb = p.ra_bias[c];
+        ib = p.ri_bias[c];
+        dc = p.decay[c];
+        yb = p.y_bias[c];
     }
-    const int blk = live ? c / block : 0;
-    const float* pre_r = pre + static_cast<int64_t>(blk) * n_tokens * 2 * block + (c - blk * block);
+    const int blk = live ? c / p.block : 0;
+    const float* pre_r = p.pre + static_cast<int64_t>(blk) * p.n_tokens * 2 * p.block + (c - blk * p.block);
     if (cluster > 1) {
         cluster_arrive_all();  // "this CTA runs": waited for before the first hand-over
     }
     pl_grid_wait();
     const int e = blockIdx.y;
-    const int start = first[e], n_all = count[e];
-    const int64_t slot = slots[e];
+    const int start = p.first[e], n_all = p.count[e];
+    const int64_t slot = p.slots[e];
     if (cluster > 1) {
         cluster_wait_all();
     }
@@ -157,12 +197,11 @@ __global__ void __launch_bounds__(kScanThreads) linear_scan_kernel(
         const int t0 = base + rank * kSpan;
         const int n = max(0, min(n_all - t0, kSpan));
         if (live) {
-#pragma unroll 4
-            for (int r = row0; r < n; r += kRowsAtOnce) {
+            for (int r = row0; r < n; r += kSubs) {
                 const int64_t t = start + t0 + r;
                 float a, b;
-                recurrence_terms<kExact>(pre_r[t * 2 * block] + rb, pre_r[t * 2 * block + block] + ib, dc,
-                                         pl_load(u + t * width + c), a, b);
+                recurrence_terms<true>(pre_r[t * 2 * p.block] + rb, pre_r[t * 2 * p.block + p.block] + ib, dc,
+                                       u[t * p.width + c], a, b);
                 a_s[r * kChannels + lane] = a;
                 b_s[r * kChannels + lane] = b;
             }
@@ -170,22 +209,8 @@ __global__ void __launch_bounds__(kScanThreads) linear_scan_kernel(
         __syncthreads();
         for (int turn = 0; turn < cluster; ++turn) {
             if (turn == rank && threadIdx.x < kChannels) {
-                float s = base == 0 && rank == 0 ? (live ? states[slot * width + c] : 0.0f) : carry[lane];
-                int r = 0;
-                for (; r + 8 <= n; r += 8) {
-                    float a[8], b[8];
-#pragma unroll
-                    for (int k = 0; k < 8; ++k) {
-                        a[k] = a_s[(r + k) * kChannels + lane];
-                        b[k] = b_s[(r + k) * kChannels + lane];
-                    }
-#pragma unroll
-                    for (int k = 0; k < 8; ++k) {
-                        s = fmaf(a[k], s, b[k]);
-                        b_s[(r + k) * kChannels + lane] = s;
-                    }
-                }
-                for (; r < n; ++r) {
+                float s = base == 0 && rank == 0 ? (live ? p.states[slot * p.width + c] : 0.0f) : carry[lane];
+                for (int r = 0; r < n; ++r) {
                     s = fmaf(a_s[r * kChannels + lane], s, b_s[r * kChannels + lane]);
                     b_s[r * kChannels + lane] = s;
                 }
@@ -204,24 +229,135 @@ __global__ void __launch_bounds__(kScanThreads) linear_scan_kernel(
             }
         }
         if (live) {
-#pragma unroll 4
-            for (int r = row0; r < n; r += kRowsAtOnce) {
+            for (int r = row0; r < n; r += kSubs) {
                 const int64_t t = start + t0 + r;
-                pl_store(out + t * width + c, b_s[r * kChannels + lane] * gelu_of<kExact>(pl_load(y + t * y_stride + c) + yb));
+                out[t * p.width + c] = b_s[r * kChannels + lane] * gelu_of<true>(y[t * p.y_stride + c] + yb);
             }
         }
         __syncthreads();
     }
-    // The first CTA was handed the state after the last token; it also moves the ring on (the convolution's kernel,
-    // which read it, has finished).
+    // (the first CTA was handed the state after the last token)
     if (rank == 0 && live && n_all > 0) {
         if (row0 == 0) {
-            states[slot * width + c] = carry[lane];
+            p.states[slot * p.width + c] = carry[lane];
         }
-        for (int j = row0; j < min(taps - 1, n_all); j += kRowsAtOnce) {
-            const int64_t t = start + n_all - 1 - j;
-            ring[(slot * taps + pos[t] % taps) * width + c] = x[t * x_stride + c];
+        move_ring_on<float>(p, c, slot, start, n_all, row0, kSubs);
+    }
+}
+
+__global__ void __launch_bounds__(kScanThreads, 2) linear_scan_composed_kernel(const ScanParams p) {
+    __shared__ float2 own_steps[kSubs][kChannels];          // this CTA's threads' steps, in token order
+    __shared__ float2 steps[2][kMaxCluster][kChannels];     // [round's parity] the CTAs' steps, in token order
+    pl_grid_trigger();
+    const int cluster = p.cluster, rank = blockIdx.x % cluster;
+    const int lane = threadIdx.x % kChannels, sub = threadIdx.x / kChannels;
+    const int c_true = (blockIdx.x / cluster) * kChannels + lane;
+    const bool live = c_true < p.width;
+    const int c = live ? c_true : p.width - 1;  // (threads past the width repeat its last channel and store nothing)
+    const __nv_bfloat16* u = static_cast<const __nv_bfloat16*>(p.u);
+    const __nv_bfloat16* y = static_cast<const __nv_bfloat16*>(p.y);
+    __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out);
+    const float rb = p.ra_bias[c], ib = p.ri_bias[c], dc = p.decay[c], yb = p.y_bias[c];
+    const int blk = c / p.block;
+    const float* pre_r = p.pre + static_cast<int64_t>(blk) * p.n_tokens * 2 * p.block + (c - blk * p.block);
+    if (cluster > 1) {
+        cluster_arrive_all();  // "this CTA runs": waited for before the first store into a peer
+    }
+    pl_grid_wait();
+    const int e = blockIdx.y;
+    const int start = p.first[e], n_all = p.count[e];
+    const int64_t slot = p.slots[e];
+    float s_base = p.states[slot * p.width + c];  // the state where the round at hand begins
+    if (cluster > 1) {
+        cluster_wait_all();
+    }
+    int round = 0;
+    for (int base = 0; base < n_all; base += cluster * kSpan, ++round) {
+        const int t0 = base + rank * kSpan + sub * kSub;
+        const int n = max(0, min(n_all - t0, kSub));
+        float a[kSub], b[kSub];
+        __nv_bfloat16 other[kSub];
+        // Loads first, a batch at a time (places past the portion's end read its last token and count for nothing).
+        constexpr int kBatch = 8;
+#pragma unroll
+        for (int i0 = 0; i0 < kSub; i0 += kBatch) {
+            if (i0 < n) {
+                float r_pre[kBatch], i_pre[kBatch];
+                __nv_bfloat16 u_in[kBatch];
+#pragma unroll
+                for (int i = 0; i < kBatch; ++i) {
+                    const int64_t t = start + min(t0 + i0 + i, n_all - 1);
+                    r_pre[i] = pre_r[t * 2 * p.block];
+                    i_pre[i] = pre_r[t * 2 * p.block + p.block];
+                    u_in[i] = u[t * p.width + c];
+                }
+#pragma unroll
+                for (int i = 0; i < kBatch; ++i) {
+                    recurrence_terms<false>(r_pre[i] + rb, i_pre[i] + ib, dc, __bfloat162float(u_in[i]), a[i0 + i], b[i0 + i]);
+                    if (i0 + i >= n) {
+                        a[i0 + i] = 1.0f;
+                        b[i0 + i] = 0.0f;
+                    }
+                }
+            } else {
+#pragma unroll
+                for (int i = 0; i < kBatch; ++i) {
+                    a[i0 + i] = 1.0f;
+                    b[i0 + i] = 0.0f;
+                }
+            }
         }
+        // (the other branch's values are asked for here, ahead of the barrier, where the terms' registers are free again)
+#pragma unroll
+        for (int i = 0; i < kSub; ++i) {
+            other[i] = y[(start + static_cast<int64_t>(min(t0 + i, n_all - 1))) * p.y_stride + c];
+        }
+        float big_a = 1.0f, big_b = 0.0f;
+#pragma unroll
+        for (int i = 0; i < kSub; ++i) {
+            big_b = fmaf(a[i], big_b, b[i]);
+            big_a *= a[i];
+        }
+        own_steps[sub][lane] = make_float2(big_a, big_b);
+        __syncthreads();
+        if (sub == 0) {
+            float2 all = own_steps[0][lane];
+            for (int k = 1; k < kSubs; ++k) {
+                const float2 step = own_steps[k][lane];
+                all = make_float2(step.x * all.x, fmaf(step.x, all.y, step.y));
+            }
+            for (int k = 0; k < cluster; ++k) {
+                cluster_store2(cluster_map(&steps[round & 1][rank][lane], k), all);
+            }
+        }
+        __syncwarp();
+        cluster_arrive_all();  // (a CTA without peers is a cluster of one)
+        cluster_wait_all();
+        float s = s_base;
+        for (int k = 0; k < cluster; ++k) {
+            s = k == rank ? s_base : s;
+            const float2 step = steps[round & 1][k][lane];
+            s_base = fmaf(step.x, s_base, step.y);
+        }
+        for (int k = 0; k < sub; ++k) {
+            const float2 step = own_steps[k][lane];
+            s = fmaf(step.x, s, step.y);
+        }
+#pragma unroll
+        for (int i = 0; i < kSub; ++i) {
+            s = fmaf(a[i], s, b[i]);
+            if (i < n && live) {
+                out[(start + static_cast<int64_t>(t0) + i) * p.width + c] =
+                    __float2bfloat16_rn(s * gelu_of<false>(__bfloat162float(other[i]) + yb));
+            }
+        }
+        __syncthreads();  // own_steps is written again (a peer writes this parity's steps again only after another barrier)
+    }
+    if (rank == 0 && live && n_all > 0) {
+        if (sub == 0) {
+            p.states[slot * p.width + c] = s_base;
+        }
+        move_ring_on<__nv_bfloat16>(p, c, slot, start, n_all, sub, kSubs);
     }
 }
 
@@ -425,14 +561,17 @@ PL_API int pl_linear_scan(const float* pre, const float* ra_bias, const float* r
     if (n_tokens == 0 || n_entries == 0) {
         return 0;
     }
+    PL_REQUIRE(dtype == PL_F32 || dtype == PL_BF16, "linear_scan: unknown dtype code %d", dtype);
     int cluster = 1;
-    while (cluster < 8 && cluster * kSpan < longest) {
+    while (cluster < kMaxCluster && cluster * kSpan < longest) {
         cluster *= 2;
     }
+    const ScanParams p = {pre, ra_bias, ri_bias, decay, u, y, y_stride, y_bias, x, x_stride, ring, taps, states,
+                          first, count, slots, pos, out, n_tokens, width, block, cluster};
     cudaLaunchConfig_t config = {};
     config.gridDim = dim3((width + kChannels - 1) / kChannels * cluster, n_entries);
     config.blockDim = dim3(kScanThreads);
-    config.dynamicSmemBytes = kScanShared;
+    config.dynamicSmemBytes = dtype == PL_F32 ? kScanShared : 0;
     config.stream = stream;
     cudaLaunchAttribute attributes[2];
     attributes[0].id = cudaLaunchAttributeClusterDimension;
@@ -444,15 +583,14 @@ PL_API int pl_linear_scan(const float* pre, const float* ra_bias, const float* r
     config.attrs = attributes;
     config.numAttrs = pl_overlap_enabled() ? 2 : 1;
     cudaError_t err = cudaSuccess;
-    PL_DISPATCH_DTYPE(dtype, "linear_scan", {
-        err = cudaFuncSetAttribute(linear_scan_kernel<scalar_t>, cudaFuncAttributeMaxDynamicSharedMemorySize, kScanShared);
+    if (dtype == PL_F32) {
+        err = cudaFuncSetAttribute(linear_scan_walked_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kScanShared);
         if (err == cudaSuccess) {
-            err = cudaLaunchKernelEx(&config, linear_scan_kernel<scalar_t>, pre, ra_bias, ri_bias, decay,
-                                     static_cast<const scalar_t*>(u), static_cast<const scalar_t*>(y), y_stride, y_bias,
-                                     static_cast<const scalar_t*>(x), x_stride, static_cast<scalar_t*>(ring), taps, states,
-                                     first, count, slots, pos, static_cast<scalar_t*>(out), n_tokens, width, block, cluster);
+            err = cudaLaunchKernelEx(&config, linear_scan_walked_kernel, p);
         }
-    });
+    } else {
+        err = cudaLaunchKernelEx(&config, linear_scan_composed_kernel, p);
+    }
     if (err != cudaSuccess) {
         return pl_fail(3, "linear_scan: launch failed: %s", cudaGetErrorString(err));
     }

@@ -12,6 +12,7 @@ import torch
 from . import native_layer
 from ..kernels import ops
 from .basic import NormedDelta, RMSNorm, ScaledPair, settle_pending
+from .branches import run_branches
 from .registry import BuildContext, build_part, register_part
 from .spec import LayerSpec
 
@@ -256,7 +257,9 @@ class ParallelBlock:
 
     def forward(self, x: torch.Tensor, delta, batch):
         tokens, hidden = x.shape
-        if self._fused() and (delta is None or isinstance(delta, ScaledPair)):
+        if self.ff_norm is None and not isinstance(delta, ScaledPair):
+            h1 = self.mixer_norm.forward(x, delta)
+        elif self._fused() and (delta is None or isinstance(delta, ScaledPair)):
             dtype, device = self.ctx.dtype, x.device
             h1 = torch.empty((tokens, hidden), dtype=dtype, device=device)
             h2 = torch.empty((tokens, hidden), dtype=dtype, device=device) if self.ff_norm is not None else None
@@ -266,14 +269,20 @@ class ParallelBlock:
                                    self.mixer_norm.eps)
         else:
             h1 = self.mixer_norm.forward(x, delta)
-            h2 = self.ff_norm.forward(x, None) if self.ff_norm is not None else None
+            h2 = self.ff_norm.forward(x, None) if self.ff_norm is not None else h1
         if self.ff_norm is None:
-            h2 = h1
+            h2 = h1   # (one norm for both sublayers)
+        if self._pending and self.feed_forward is None:
+            return x, self.mixer.pending(h1, batch)
         if self._pending:
-            sides = self.mixer.pending(h1, batch)
-            return x, sides.with_third(self.feed_forward.forward(h2, batch) if self.feed_forward is not None else None)
-        y1 = self.mixer.forward(h1, batch)
-        y2 = self.feed_forward.forward(h2, batch) if self.feed_forward is not None else None
+            sides, third = run_branches(batch, x.device, lambda: self.mixer.pending(h1, batch),
+                                        feed_forward=lambda: self.feed_forward.forward(h2, batch))
+            return x, sides.with_third(third)
+        if self.feed_forward is None:
+            y1, y2 = self.mixer.forward(h1, batch), None
+        else:
+            y1, y2 = run_branches(batch, x.device, lambda: self.mixer.forward(h1, batch),
+                                  feed_forward=lambda: self.feed_forward.forward(h2, batch))
         return x, ScaledPair(y1, self.scales.mixer, y2, self.scales.feed_forward)
 
 

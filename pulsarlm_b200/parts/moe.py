@@ -8,6 +8,7 @@ import os
 import torch
 
 from ..kernels import ops
+from .branches import run_branches
 from .linear import activated_linear, gated_feed_forward, linear
 from .registry import BuildContext, Part, register_part
 from .spec import PartSpec, TensorNeed
@@ -130,39 +131,53 @@ class RoutedExperts(Part):
         return (h.dtype == torch.bfloat16 and h.shape[0] >= GROUPED_MIN_TOKENS and self.hidden % 8 == 0
                 and self.ff % 8 == 0 and hasattr(torch.nn.functional, "grouped_mm"))
 
-    def forward(self, h: torch.Tensor, batch) -> torch.Tensor:
-        tokens = h.shape[0]
-        shared_weights = torch.empty(tokens, dtype=torch.float32, device=h.device) if self.shared_gate_row else None
+    def _route(self, h: torch.Tensor) -> tuple:
+        """(ids, weights on the experts' inputs, weights on their outputs, weight of the shared expert); weights None: 1."""
+        shared = torch.empty(h.shape[0], dtype=torch.float32, device=h.device) if self.shared_gate_row else None
         ids, weights = ops.moe_route(h, self.router, self.correction, self.top, self.groups, self.keep,
-                                     self.sigmoid_scores, self.group_top, self.renormalise, shared_weights)
-        in_weights, out_weights = (weights, None) if self.weigh_input else (None, weights)
-        shared = None
-        if self.shared_size and self.gated:
-            act = "silu" if self.shared_limit is None else "clamped"
-            shared = gated_feed_forward(h, self.shared_gate_up, self.shared_down, act, self.shared_limit or 0.0)
-        elif self.shared_size:
-            shared = activated_linear(linear(h, self.shared_gate_up), None, "relu2", self.shared_down)
-        out = torch.empty((tokens, self.hidden), dtype=h.dtype, device=h.device)
-        if self._grouped(h):
-            # Pairs in expert order; each projection one grouped product over the sorted rows (the
-            # library's: operands [rows, K] and [E, K, N] with the experts' last rows as offsets).
-            ends, row_of_pair, pair_of_row = ops.moe_sort(ids, self.n_experts)
-            x = ops.moe_gather(h, pair_of_row, self.top)
-            gate_up = torch.nn.functional.grouped_mm(x, self.gate_up.transpose(1, 2), offs=ends)
-            act = torch.empty((x.shape[0], self.ff), dtype=h.dtype, device=h.device)
-            if self.limit is not None:
-                ops.gated_act(gate_up, act, "clamped", self.limit, in_weights, pair_of_row)
-            elif self.gated:
-                ops.swiglu(gate_up, act)
-            else:
-                ops.bias_act(gate_up, None, act, "relu2")
-            y = torch.nn.functional.grouped_mm(act, self.down.transpose(1, 2), offs=ends)
-            ops.moe_combine(y, row_of_pair, out_weights, shared, out, shared_weights)
-            return out
-        act = torch.empty((tokens * self.top, self.ff), dtype=h.dtype, device=h.device)
+                                     self.sigmoid_scores, self.group_top, self.renormalise, shared)
+        return (ids, weights, None, shared) if self.weigh_input else (ids, None, weights, shared)
+
+    def _shared(self, h: torch.Tensor) -> torch.Tensor | None:
+        """The shared expert's output."""
+        if not self.shared_size:
+            return None
         if self.gated:
-            ops.moe_gate_up(h, self.gate_up, ids, act, self.limit, in_weights)
+            act = "silu" if self.shared_limit is None else "clamped"
+            return gated_feed_forward(h, self.shared_gate_up, self.shared_down, act, self.shared_limit or 0.0)
+        return activated_linear(linear(h, self.shared_gate_up), None, "relu2", self.shared_down)
+
+    def _units(self, h: torch.Tensor) -> tuple:
+        """Router and first half of the chosen experts, pair by pair: (activations [T * top, F], what `_route` says)."""
+        routed = self._route(h)
+        act = torch.empty((h.shape[0] * self.top, self.ff), dtype=h.dtype, device=h.device)
+        if self.gated:
+            ops.moe_gate_up(h, self.gate_up, routed[0], act, self.limit, routed[1])
         else:
-            ops.moe_up(h, self.gate_up, ids, act)
-        ops.moe_down(act, self.down, ids, out_weights, shared, out, shared_weights)
+            ops.moe_up(h, self.gate_up, routed[0], act)
+        return act, routed
+
+    def forward(self, h: torch.Tensor, batch) -> torch.Tensor:
+        out = torch.empty((h.shape[0], self.hidden), dtype=h.dtype, device=h.device)
+        if not self._grouped(h):
+            (act, (ids, _, weights, shared_weights)), shared = run_branches(
+                batch, h.device, lambda: self._units(h), shared_expert=lambda: self._shared(h))
+            ops.moe_down(act, self.down, ids, weights, shared, out, shared_weights)
+            return out
+        # Pairs in expert order; each projection one grouped product over the sorted rows (the library's: operands
+        # [rows, K] and [E, K, N] with the experts' last rows as offsets).
+        ids, in_weights, weights, shared_weights = self._route(h)
+        shared = self._shared(h)
+        ends, row_of_pair, pair_of_row = ops.moe_sort(ids, self.n_experts)
+        x = ops.moe_gather(h, pair_of_row, self.top)
+        gate_up = torch.nn.functional.grouped_mm(x, self.gate_up.transpose(1, 2), offs=ends)
+        act = torch.empty((x.shape[0], self.ff), dtype=h.dtype, device=h.device)
+        if self.limit is not None:
+            ops.gated_act(gate_up, act, "clamped", self.limit, in_weights, pair_of_row)
+        elif self.gated:
+            ops.swiglu(gate_up, act)
+        else:
+            ops.bias_act(gate_up, None, act, "relu2")
+        y = torch.nn.functional.grouped_mm(act, self.down.transpose(1, 2), offs=ends)
+        ops.moe_combine(y, row_of_pair, weights, shared, out, shared_weights)
         return out

@@ -6,6 +6,7 @@ import torch
 
 from ..kernels import ops
 from .basic import NormedSides
+from .branches import run_branches
 from .linear import linear
 from .registry import BuildContext, Part, build_part, part_class, register_part
 from .spec import PartSpec, TensorNeed
@@ -80,8 +81,9 @@ class SideBySide(Part):
         """Both mixers' outputs as a residual contribution that is normed on its way in."""
         proj = linear(h, self.in_weight)
         at, stride = self.left.channels, self.in_weight.shape[0]
-        left = self.left.forward_columns(proj[:, :at], stride, h, batch, True)
-        right = self.right.forward_columns(proj[:, at:], stride, h, batch, True)
+        left, right = run_branches(batch, h.device,
+                                   lambda: self.left.forward_columns(proj[:, :at], stride, h, batch, True),
+                                   right=lambda: self.right.forward_columns(proj[:, at:], stride, h, batch, True))
         return NormedSides(left, self.left.output_bias, self.left_weight, right, self.right.output_bias, self.right_weight,
                            0.5, self.eps)
 
