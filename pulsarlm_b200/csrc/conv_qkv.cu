@@ -9,8 +9,8 @@
 // paged attention kernels know; a product with a zero adds nothing. Earlier inputs of a sequence come from the step's
 // own rows where the portion has them and from the request's state slot where not (the slot holds the last taps - 1
 // projected rows, without the bias, as the product wrote them). In a step whose entries bring one token each the slot
-// moves on in the same launch (every channel belongs to one thread); otherwise the caller updates it afterwards
-// (short_conv.cu). Everything is fp32 with one rounding on each store, the taps in order from the oldest.
+// moves on in the same launch (every channel belongs to one thread); otherwise a second kernel moves it on afterwards
+// (pl_filter_state). Everything is fp32 with one rounding on each store, the taps in order from the oldest.
 //
 // A thread takes a piece of a row (16 bytes where sizes and addresses allow, else one element) for a few
 // neighbouring tokens; with few taps (known to the compiler) the earlier inputs stay in registers from token to token.
@@ -192,6 +192,31 @@ __global__ void __launch_bounds__(kThreads) conv_qkv_write_kernel(const ConvQkvP
     }
 }
 
+// The slots after the step, one block row per entry: row j becomes the input `taps - 1 - j` places before the next token,
+// from the step's rows or, for a portion shorter than that, moved up inside the slot (a thread owns a piece of every
+// row and walks them upwards, so it reads a row before it writes it).
+template <typename scalar_t, int PER>
+__global__ void __launch_bounds__(kThreads) filter_state_kernel(
+        const scalar_t* __restrict__ proj, int64_t row_stride, const int32_t* __restrict__ first,
+        const int32_t* __restrict__ count, const int32_t* __restrict__ slots, scalar_t* __restrict__ state, int reach,
+        int channels) {
+    using Piece = RowPiece<scalar_t, PER>;
+    pl_grid_trigger();
+    pl_grid_wait();
+    const int c = (blockIdx.x * kThreads + threadIdx.x) * PER;
+    if (c >= channels) {
+        return;
+    }
+    const int e = blockIdx.y, n = count[e];
+    scalar_t* mine = state + static_cast<int64_t>(slots[e]) * reach * channels + c;
+    const scalar_t* rows = proj + static_cast<int64_t>(first[e]) * row_stride + c;
+    for (int j = 0; j < reach; ++j) {
+        const int at = n - reach + j;  // among the portion's rows
+        Piece::put(mine + static_cast<int64_t>(j) * channels,
+                   at >= 0 ? Piece::get(rows + at * row_stride) : Piece::get(mine + static_cast<int64_t>(n + j) * channels));
+    }
+}
+
 template <typename scalar_t, int PER>
 void launch(const ConvQkvParams& p, cudaStream_t stream) {
     const int pieces = (p.n_heads + 2 * p.n_kv) * (p.row / PER);
@@ -276,5 +301,36 @@ PL_API int pl_conv_qkv_write(const void* proj, int64_t row_stride, const float* 
         return pl_fail(2, "conv_qkv_write: unknown dtype code %d", dtype);
     }
     PL_CHECK_LAUNCH("conv_qkv_write");
+    return 0;
+}
+
+// Brings every entry's slot of the state [slots, taps - 1, channels] up to date with the step's rows (run after
+// pl_conv_qkv_write has read the old slots): first, count int32 [entries], the row of each entry's first token and how
+// many it brings.
+PL_API int pl_filter_state(const void* proj, int64_t row_stride, const int32_t* first, const int32_t* count,
+                           const int32_t* slots, void* state, int n_entries, int channels, int taps, int dtype,
+                           cudaStream_t stream) {
+    PL_REQUIRE(n_entries >= 0 && n_entries <= 65535 && channels > 0 && taps >= 1 && row_stride >= channels,
+               "filter_state: bad sizes entries=%d channels=%d taps=%d", n_entries, channels, taps);
+    if (n_entries == 0 || taps == 1) {
+        return 0;
+    }
+    const int per = dtype == PL_F32 ? 4 : 8;
+    const bool pieces = channels % per == 0 && row_stride % per == 0 &&
+        ((reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(state)) & 15) == 0;
+    const int lanes = pieces ? channels / per : channels;
+    const dim3 grid((lanes + kThreads - 1) / kThreads, n_entries);
+#define PL_FILTER_STATE(S, PER)                                                                                       \
+    pl_launch_overlapped(filter_state_kernel<S, PER>, grid, dim3(kThreads), 0, stream, static_cast<const S*>(proj),   \
+                         row_stride, first, count, slots, static_cast<S*>(state), taps - 1, channels)
+    if (dtype == PL_F32) {
+        if (pieces) { PL_FILTER_STATE(float, 4); } else { PL_FILTER_STATE(float, 1); }
+    } else if (dtype == PL_BF16) {
+        if (pieces) { PL_FILTER_STATE(__nv_bfloat16, 8); } else { PL_FILTER_STATE(__nv_bfloat16, 1); }
+    } else {
+        return pl_fail(2, "filter_state: unknown dtype code %d", dtype);
+    }
+#undef PL_FILTER_STATE
+    PL_CHECK_LAUNCH("filter_state");
     return 0;
 }

@@ -34,8 +34,9 @@ __device__ __forceinline__ float gate_activation(float z, int act) {
     return z / (1.0f + expf(-z));
 }
 
+template <bool EXACT>
 __device__ __forceinline__ float gate_unit(float g, float u, float w, const GateParams& p) {
-    return p.act == 2 ? pl_clamped_unit(w * g, w * u, p.limit) : gate_activation(g, p.act) * u;
+    return p.act == 2 ? pl_clamped_unit<EXACT>(w * g, w * u, p.limit) : gate_activation(g, p.act) * u;
 }
 __device__ __forceinline__ float row_weight(const GateParams& p, int64_t t) {
     return p.row_weights == nullptr ? 1.0f : p.row_weights[p.row_index != nullptr ? p.row_index[t] : t];
@@ -55,8 +56,8 @@ __global__ void gated_act_kernel(const scalar_t* __restrict__ in, scalar_t* __re
         const float4 g = pl_load4(in + t * 2 * width + i);
         const float4 u = pl_load4(in + t * 2 * width + width + i);
         const float w = row_weight(p, t);
-        pl_store4(out + t * width + i, make_float4(gate_unit(g.x, u.x, w, p), gate_unit(g.y, u.y, w, p),
-                                                   gate_unit(g.z, u.z, w, p), gate_unit(g.w, u.w, w, p)));
+        pl_store4(out + t * width + i, make_float4(gate_unit<sizeof(scalar_t) == 4>(g.x, u.x, w, p), gate_unit<sizeof(scalar_t) == 4>(g.y, u.y, w, p),
+                                                   gate_unit<sizeof(scalar_t) == 4>(g.z, u.z, w, p), gate_unit<sizeof(scalar_t) == 4>(g.w, u.w, w, p)));
     }
 }
 
@@ -70,7 +71,7 @@ __global__ void gated_act_scalar_kernel(const scalar_t* __restrict__ in, scalar_
          idx += static_cast<int64_t>(gridDim.x) * blockDim.x) {
         const int64_t t = idx / width;
         const int i = static_cast<int>(idx - t * width);
-        pl_store(out + idx, gate_unit(pl_load(in + t * 2 * width + i), pl_load(in + t * 2 * width + width + i),
+        pl_store(out + idx, gate_unit<sizeof(scalar_t) == 4>(pl_load(in + t * 2 * width + i), pl_load(in + t * 2 * width + width + i),
                                       row_weight(p, t), p));
     }
 }

@@ -30,7 +30,7 @@
 // the 64 up rows of the same features (two TMA boxes per stage); in the epilogue the
 // warps that hold the up rows pass them through shared memory to the warps that hold
 // the gate rows, which round both to bfloat16 (as a product that stored them would)
-// and apply the activation.
+// and apply the activation (or the clamped unit of gate_units.cuh: a build of its own).
 //
 // Every wait on an mbarrier is bounded: after the limit the CTA raises bit 8 of the
 // status word, stops issuing work, lets what is in flight land, meets its partner,
@@ -38,6 +38,7 @@
 //
 // The reference leaves these products to a library (`at::linear`,
 // pulsarlm-core/src/engine/model/llama.cpp:67-69, 81, 91, 93).
+#include "gate_units.cuh"
 #include "tcgen05_helpers.cuh"
 
 namespace {
@@ -56,6 +57,7 @@ struct PairParams {
     int t, n, k;  // n: output features (gated: W has 2n rows)
     int64_t ldy;
     int out_f32;
+    float limit;  // (the clamped unit)
     int n_tiles;  // tiles along N (256 features each)
     int t_tiles;  // tiles along T (256 tokens each)
     int k_blocks;
@@ -114,7 +116,8 @@ __device__ __forceinline__ void arrive_on_first(uint64_t* bar) {
 constexpr int kGateRow = 17;  // 16 token columns handed over per thread and chunk, padded against bank conflicts
 constexpr int kGateBytes = 2 * 2 * (kTileM / 2) * kGateRow * 4;  // two buffers of [gate side, up side][64][17] floats
 
-template <bool GATED>
+// GATED: 0 the product alone, 1 silu(gate) * up, 2 the clamped unit of gate and up.
+template <int GATED>
 __global__ void __launch_bounds__(kThreads, 1)
 gemm_pair_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x,
                  const PairParams p) {
@@ -286,7 +289,7 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
                             // both products rounded as a product that stored them would round them
                             const float g = __bfloat162float(__float2bfloat16_rn(is_up ? other[c] : own));
                             const float u = __bfloat162float(__float2bfloat16_rn(is_up ? own : other[c]));
-                            act[c] = __fdividef(g, 1.0f + __expf(-g)) * u;
+                            act[c] = GATED == 2 ? pl_clamped_unit<false>(g, u, p.limit) : __fdividef(g, 1.0f + __expf(-g)) * u;
                         }
 #pragma unroll
                         for (int c = 0; c < 16; ++c) {
@@ -368,7 +371,7 @@ PL_API int pl_gemm_bf16_pair_supports(int t, int n, int k, int64_t ldx, int64_t 
 
 namespace {
 
-template <bool GATED>
+template <int GATED>
 int launch_pair(const CUtensorMap& map_w, const CUtensorMap& map_x, const PairParams& p, int used_pairs,
                 cudaStream_t stream) {
     constexpr int smem = kStages * kStageBytes + (GATED ? kGateBytes : 0) + 1024;
@@ -409,8 +412,8 @@ int launch_pair(const CUtensorMap& map_w, const CUtensorMap& map_x, const PairPa
 // `gated`, w is [2N, K] (a gate matrix over an up matrix) and
 // y = silu(x gate^T) * (x up^T), both products rounded to bfloat16 first (a tile is
 // then 128 output features x 256 tokens).
-PL_API int pl_gemm_bf16_pair(const void* x, const void* w, void* y, int t, int n, int k, int64_t ldx, int64_t ldw,
-                             int64_t ldy, int out_f32, int gated, int32_t* status, cudaStream_t stream) {
+static int run_pair(const void* x, const void* w, void* y, int t, int n, int k, int64_t ldx, int64_t ldw, int64_t ldy,
+                    int out_f32, int gated, float limit, int32_t* status, cudaStream_t stream) {
     PL_REQUIRE(pl_gemm_bf16_pair_supports(t, n, k, ldx, ldw),
                "gemm_bf16_pair: unsupported sizes t=%d n=%d k=%d ldx=%lld ldw=%lld (k and the leading dimensions "
                "must be multiples of 8)",
@@ -434,12 +437,25 @@ PL_API int pl_gemm_bf16_pair(const void* x, const void* w, void* y, int t, int n
     p.k = k;
     p.ldy = ldy;
     p.out_f32 = out_f32;
+    p.limit = limit;
     p.n_tiles = (n + per_pair - 1) / per_pair;
     p.t_tiles = (t + kPairN - 1) / kPairN;
     p.k_blocks = (k + kBlockK - 1) / kBlockK;
     p.total_tiles = p.n_tiles * p.t_tiles;
     const int used_pairs = p.total_tiles < pair_count() ? p.total_tiles : pair_count();
     p.status = status;
-    return gated ? launch_pair<true>(map_w, map_x, p, used_pairs, stream)
-                 : launch_pair<false>(map_w, map_x, p, used_pairs, stream);
+    return gated == 2 ? launch_pair<2>(map_w, map_x, p, used_pairs, stream)
+        : gated       ? launch_pair<1>(map_w, map_x, p, used_pairs, stream)
+                      : launch_pair<0>(map_w, map_x, p, used_pairs, stream);
+}
+
+PL_API int pl_gemm_bf16_pair(const void* x, const void* w, void* y, int t, int n, int k, int64_t ldx, int64_t ldw,
+                             int64_t ldy, int out_f32, int gated, int32_t* status, cudaStream_t stream) {
+    return run_pair(x, w, y, t, n, k, ldx, ldw, ldy, out_f32, gated != 0, 0.0f, status, stream);
+}
+
+// Gated, with the clamped unit (gate_units.cuh) of the two rounded products in the place of silu(gate) * up.
+PL_API int pl_gemm_bf16_pair_clamped(const void* x, const void* w, void* y, int t, int n, int k, int64_t ldx, int64_t ldw,
+                                     int64_t ldy, int out_f32, float limit, int32_t* status, cudaStream_t stream) {
+    return run_pair(x, w, y, t, n, k, ldx, ldw, ldy, out_f32, 2, limit, status, stream);
 }

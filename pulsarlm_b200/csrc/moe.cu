@@ -411,7 +411,7 @@ __global__ void moe_gate_up_kernel(const scalar_t* __restrict__ h, int64_t h_str
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
     const float in_weight = CLAMPED && in_weights != nullptr ? in_weights[pair] : 1.0f;
     auto unit = [&](float g, float u) {
-        return CLAMPED ? pl_clamped_unit(in_weight * g, in_weight * u, limit) : silu_f32(g) * u;
+        return CLAMPED ? pl_clamped_unit<sizeof(scalar_t) == 4>(in_weight * g, in_weight * u, limit) : silu_f32(g) * u;
     };
     for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
         row[i] = pl_load(h + t * h_stride + i);

@@ -25,7 +25,7 @@ _PTR = ctypes.c_void_p
 _lib = None
 _lock = threading.Lock()
 
-ABI_VERSION = 29
+ABI_VERSION = 30
 
 DTYPE_CODE = {torch.float32: 0, torch.bfloat16: 1}
 
@@ -87,6 +87,7 @@ _SIGNATURES = {
     "pl_gemm_bf16_skinny": [_PTR, _PTR, _PTR, _I32, _I32, _I32, _I64, _I64, _I64, _I32, _PTR, _PTR],
     "pl_gemm_bf16_skinny_max_tokens": [],
     "pl_gemm_bf16_pair": [_PTR, _PTR, _PTR, _I32, _I32, _I32, _I64, _I64, _I64, _I32, _I32, _PTR, _PTR],
+    "pl_gemm_bf16_pair_clamped": [_PTR, _PTR, _PTR, _I32, _I32, _I32, _I64, _I64, _I64, _I32, _F32, _PTR, _PTR],
     "pl_attention_decode_resident_clusters": [_I32, _I32, _I32],
     "pl_gemm_bf16_skinny_splits": [_I32, _I32, _I32],
     "pl_pair_residual_norm": [_PTR, _PTR, _PTR, _PTR, _PTR, _PTR, _PTR, _PTR, _PTR, _PTR, _PTR, _I32, _I32, _F32, _I32,
@@ -127,6 +128,7 @@ _SIGNATURES = {
     "pl_conv_qkv_write": [_PTR, _I64, _PTR, _PTR, _I32, _PTR, _PTR, _I32, _I32, _F32, _I32, _PTR, _PTR, _PTR, _I32, _PTR,
                           _PTR, _PTR, _I64, _I64, _I32, _I32, _I32, _I32, _I32, _I32, _I32, _I32, _I32, _I32, _I32, _PTR,
                           _PTR],
+    "pl_filter_state": [_PTR, _I64, _PTR, _PTR, _PTR, _PTR, _I32, _I32, _I32, _I32, _PTR],
     "pl_ring_conv": [_PTR, _I64, _PTR, _PTR, _PTR, _I32, _PTR, _PTR, _PTR, _PTR, _PTR, _PTR, _I32, _I32, _I32, _PTR],
     "pl_linear_scan": [_PTR, _PTR, _PTR, _PTR, _PTR, _PTR, _I64, _PTR, _PTR, _I64, _PTR, _I32, _PTR, _PTR, _PTR, _PTR,
                        _PTR, _PTR, _I32, _I32, _I32, _I32, _I32, _I32, _PTR],
@@ -920,6 +922,19 @@ def conv_qkv_write(proj: torch.Tensor, row_stride: int, bias: torch.Tensor | Non
           n_heads, n_kv, dim, vdim, row, k_col, v_col, _code(proj.dtype), _p(status), _stream())
 
 
+def filter_state(proj: torch.Tensor, row_stride: int, first: torch.Tensor, count: torch.Tensor, slots: torch.Tensor,
+                 state: torch.Tensor) -> None:
+    """Brings every entry's slot of state [slots, taps - 1, channels] up to date with the step's projected rows proj [T,
+    channels] (`row_stride` elements apart); first, count int32 [entries]. After conv_qkv_write has read the slots."""
+    _dev(proj, first, count, slots, state)
+    assert proj.stride(1) == 1 and (proj.shape[0] == 1 or proj.stride(0) == row_stride) and state.dtype == proj.dtype
+    assert state.is_contiguous() and state.shape[2] == proj.shape[1]
+    for t in (first, count, slots):
+        assert t.dtype == torch.int32 and t.is_contiguous()
+    _call("pl_filter_state", _p(proj), int(row_stride), _p(first), _p(count), _p(slots), _p(state), first.numel(),
+          proj.shape[1], state.shape[1] + 1, _code(proj.dtype), _stream())
+
+
 def ring_conv(x: torch.Tensor, row_stride: int, x_bias: torch.Tensor, weight: torch.Tensor, conv_bias: torch.Tensor,
               ring: torch.Tensor, first: torch.Tensor, entry: torch.Tensor, slots: torch.Tensor, pos: torch.Tensor,
               out: torch.Tensor) -> None:
@@ -1045,7 +1060,7 @@ GEMM_SKINNY_MAX_TOKENS = 64
 
 
 def gemm_bf16(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, status: torch.Tensor | None = None,
-              kernel: str | None = None, gated: bool = False) -> None:
+              kernel: str | None = None, gated: bool = False, limit: float | None = None) -> None:
     """out[T, N] (bf16 or fp32) = x[T, K] @ w[N, K]^T on the tcgen05 tensor cores.
 
     Two kernels: "skinny" for up to 64 tokens (one tile and part of k per CTA, the parts
@@ -1053,7 +1068,8 @@ def gemm_bf16(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, status: torch
     any token count, meant for prompts). `kernel=None` picks by the token count.
 
     gated (pair only): w is [2N, K], a gate matrix over an up matrix, and
-    out = silu(x gate^T) * (x up^T), both products rounded to bfloat16 first."""
+    out = silu(x gate^T) * (x up^T), both products rounded to bfloat16 first; with `limit` the
+    clamped unit of the two (csrc/gate_units.cuh) instead."""
     _dev(x, w, out, status)
     assert x.dtype == w.dtype == torch.bfloat16 and out.dtype in (torch.bfloat16, torch.float32)
     t, k = x.shape
@@ -1068,6 +1084,10 @@ def gemm_bf16(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, status: torch
         assert not gated, "only the pair kernel has the gated epilogue"
         _call("pl_gemm_bf16_skinny", _p(x), _p(w), _p(out), t, n, k, ldx, ldw, out.stride(0) if t > 1 else n,
               int(out.dtype == torch.float32), _p(status), _stream())
+        return
+    if kernel == "pair" and gated and limit is not None:
+        _call("pl_gemm_bf16_pair_clamped", _p(x), _p(w), _p(out), t, n, k, ldx, ldw, out.stride(0) if t > 1 else n,
+              int(out.dtype == torch.float32), float(limit), _p(status), _stream())
         return
     if kernel == "pair":
         _call("pl_gemm_bf16_pair", _p(x), _p(w), _p(out), t, n, k, ldx, ldw, out.stride(0) if t > 1 else n,

@@ -9,6 +9,7 @@ import torch
 
 from ..kernels import ops
 from .attention import Attention
+from .delta_rule import sequence_rows_plan
 from .gated_delta import FilterState
 from .linear import linear
 from .registry import BuildContext, register_part
@@ -142,6 +143,14 @@ class FilteredAttention(Attention):
     def captures_state_steps(self) -> bool:
         return True
 
+    def plan_key(self):
+        key = super().plan_key()
+        return ("filtered", *key) if key is not None else None
+
+    def plan_step(self, step) -> dict:
+        """What attention plans, and the rows of every entry (for the convolutions' slots)."""
+        return {**super().plan_step(step), **sequence_rows_plan(step)}
+
     def _folds_rope(self, tokens, batch, inv_freq, rotary) -> bool:
         return False  # (nothing is rotated; the convolution is a kernel of its own)
 
@@ -164,7 +173,8 @@ class FilteredAttention(Attention):
                            self.temp_every, batch.pos, batch.entry, table, q, cache.k_pool, cache.v_pool, cache.page_size,
                            self.n_kv, self.key_dim, self.value_dim, self.starts[1], self.starts[2], batch.status)
         if self.taps > 1 and not single:
-            ops.short_conv_state_strided(proj, batch.entry, batch.slots, states)
+            plan = batch.plans[self.plan_key()]
+            ops.filter_state(proj, row_stride, plan["first"], plan["count"], batch.slots, states)
         out = torch.empty((tokens, self.n_heads, self.row), dtype=proj.dtype, device=proj.device)
         self.attend(q, out, table, batch)
         y = linear(out.view(tokens, self.n_heads * self.row), self.o)

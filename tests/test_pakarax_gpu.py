@@ -99,7 +99,9 @@ def test_filtered_queries_keys_and_values_on_the_way_to_the_cache(heads, kv, dim
                            _i32(pos), entry_t, table[[r for r, _ in step]].to(DEV), q, k_pool, v_pool, page, kv, dim, vdim,
                            starts[1], starts[2])
         if taps > 1 and not single:
-            ops.short_conv_state_strided(proj[:, :width], entry_t, slots_t, state)
+            counts = [entry.count(e) for e in range(len(step))]
+            firsts = [sum(counts[:e]) for e in range(len(step))]
+            ops.filter_state(proj[:, :width], width + 8, _i32(firsts), _i32(counts), slots_t, state)
         want_q = torch.stack([want[step[e][0]][0][p] for e, p in zip(entry, pos)])
         assert plain.relative_error_of(q[:, :, :dim].cpu(), want_q) < bar, step
         assert row == dim or float(q[:, :, dim:].abs().max()) == 0.0
@@ -495,6 +497,21 @@ def test_gated_feed_forward_with_the_clamped_unit(tokens, dtype):
     d = {k: v.double() for k, v in w.items()}
     want = plain.clamped_ff(h.double(), d["gate"], d["up"], d["down"], 0.9, lambda t: t)
     assert plain.relative_error_of(part.forward(h.to(DEV), None).cpu(), want) < (1e-5 if dtype == "float32" else 2e-2)
+
+
+@pytest.mark.parametrize("tokens,ff", [(300, 200), (257, 136), (64, 512)])
+def test_clamped_unit_in_the_epilogue_of_a_prompt_product(tokens, ff):
+    """The pair kernel forms the unit from the rounded products, as the kernel alone does."""
+    ops = _ops()
+    gen = torch.Generator().manual_seed(ff)
+    width, limit, bf = 96, 0.8, torch.bfloat16
+    x = torch.randn(tokens, width, generator=gen).to(bf)
+    gate_up = (2.0 * torch.randn(2 * ff, width, generator=gen) / width ** 0.5).to(bf)
+    both = (x.double() @ gate_up.double().T).to(bf).double()
+    want = plain.clamped_unit(both[:, :ff], both[:, ff:], limit)
+    act = torch.empty(tokens, ff, dtype=bf, device=DEV)
+    ops.gemm_bf16(x.to(DEV), gate_up.to(DEV), act, kernel="pair", gated=True, limit=limit)
+    assert plain.relative_error_of(act.cpu(), want) < 1e-2
 
 
 def test_scaled_and_capped_logits():
