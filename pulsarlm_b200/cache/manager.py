@@ -1,13 +1,14 @@
 """The cache manager: paged keys and values per layer group, block tables per
 request, and fixed-size state slots.
 
-Layers whose mixers ask for the same KVCacheNeed (kv heads, head size, window)
+Layers whose mixers ask for the same KVCacheNeed (kv heads, head size, window, kept first tokens)
 form a group. A group has its own page pool: one tensor
 [layers in group, pages + 1, 2 (K, V), kv heads, page size, head size] (the last
 page is never handed out: padding rows of captured steps use it), so one page
 id holds `page_size` tokens of every layer of the group, and a request has one
 block table per group. Groups with a window give pages back as soon as every
-token in them is out of every future query's reach, and when the caller bounds
+token in them is out of every future query's reach (a group that keeps a sequence's
+first tokens in reach keeps their pages), and when the caller bounds
 the tokens a request brings to one step their pools are made only as large as
 `max_requests` such requests can fill (`window_pages`). Mixers that ask for a
 StateNeed get a row per request slot in a tensor [slots, *shape], zeroed when
@@ -87,14 +88,15 @@ def flat_needs(needs: list) -> list[tuple]:
     return out
 
 
-def window_pages(window: int, page_size: int, step_tokens: int, max_requests: int) -> int:
+def window_pages(window: int, page_size: int, step_tokens: int, max_requests: int, keep_first: int = 0) -> int:
     """Pages that `max_requests` requests can hold at once in a group whose queries
     reach `window` keys back, when no request brings more than `step_tokens` tokens to
     a step. A request of length L that reserves n more tokens holds the pages from
     that of key L - window + 1 to that of key L + n - 1: fewer than
     (window + n - 1) / page_size + 2. One token more, for a step that is reserved
-    while the step before it has not been committed."""
-    per_request = -(-(window + step_tokens + 1) // page_size) + 1
+    while the step before it has not been committed. The pages of `keep_first` tokens at the
+    sequence's start come on top."""
+    per_request = -(-(window + step_tokens + 1) // page_size) + 1 + -(-keep_first // page_size)
     return max_requests * per_request
 
 
@@ -102,7 +104,7 @@ def pool_pages(need: KVCacheNeed, n_pages: int, page_size: int, step_tokens: int
     """Pages of the pool of a group with this need, when groups that keep every key get n_pages."""
     if need.window is None or step_tokens is None:
         return n_pages
-    return min(n_pages, window_pages(need.window, page_size, step_tokens, max_requests))
+    return min(n_pages, window_pages(need.window, page_size, step_tokens, max_requests, need.keep_first))
 
 
 def cache_bytes(needs: list, n_pages: int, page_size: int, step_tokens: int | None, max_requests: int,
@@ -191,8 +193,9 @@ class CacheManager:
         self._lib = core.library()
         windows = (ctypes.c_int32 * max(1, len(self.groups)))(
             *[g.need.window if g.need.window is not None else -1 for g in self.groups])
+        kept = (ctypes.c_int32 * max(1, len(self.groups)))(*[g.need.keep_first for g in self.groups])
         pages = (ctypes.c_int32 * max(1, len(self.groups)))(*[g.n_pages for g in self.groups])
-        self._book = self._lib.plh_cache_create(len(self.groups), windows, page_size, pages, max_requests,
+        self._book = self._lib.plh_cache_create(len(self.groups), windows, kept, page_size, pages, max_requests,
                                                 int(mass_decay is not None))
         for group in self.groups:
             group.pool = GroupPoolView(self._lib, self._book, group.index, group.n_pages)

@@ -97,6 +97,7 @@ struct DecodeParams {
     const float* distance_bias;  // fp32 [n_heads, bias_rows] (nullptr: none), see PlAttentionExtras
     int bias_rows;
     const float* distance_slopes;  // fp32 [n_heads] (nullptr: none)
+    int keep_first;  // the request's first keys that stay in reach besides the window's (not in work-list mode)
 };
 
 // In-cluster merge: outputs are counted in groups of four dims ("vecs"); rank r owns
@@ -147,7 +148,13 @@ __device__ __forceinline__ void attention_decode_share(const DecodeParams& p, un
     }
     const int ctx = p.pos[t] + 1;
     const int first = p.window > 0 ? max(0, ctx - p.window) : 0;
-    const int tile_first = first / kTile, tile_end = (ctx + kTile - 1) / kTile;
+    // Tiles are counted by their place in the walk (with kept first keys it jumps from their tiles to the
+    // window's; without, and over a work list, a place is the tile itself).
+    const int keep = EXTRAS && p.items == nullptr ? p.keep_first : 0;
+    const PlTileWalk walk(first, keep, kTile);
+    const int shift = keep > 0 ? walk.start - walk.head : 0;  // tile = place, or place + shift past the kept keys' tiles
+    const int tile_first = keep > 0 ? 0 : first / kTile, tile_end = (ctx + kTile - 1) / kTile - shift;
+    auto tile_at = [&](int place) { return EXTRAS && place >= walk.head ? place + shift : place; };
     const int per_split = p.items != nullptr ? item_tiles : (tile_end - tile_first + n_splits - 1) / n_splits;
     const int t0 = p.items != nullptr ? item_first : tile_first + split * per_split;
     const int t1 = min(t0 + per_split, tile_end);
@@ -168,7 +175,7 @@ __device__ __forceinline__ void attention_decode_share(const DecodeParams& p, un
         if (i % 32 == 0 && i < my_tiles) {
             // one coalesced look-up of the block table for the next 32 tiles
             const int mine = i + lane;
-            my_page = mine < my_tiles ? row[((t0 + warp + mine * WARPS) * kTile) / p.page_size] : 0;
+            my_page = mine < my_tiles ? row[(tile_at(t0 + warp + mine * WARPS) * kTile) / p.page_size] : 0;
             if (my_page < 0 || my_page >= p.n_pages) {
                 if (p.status != nullptr) {
                     atomicOr(p.status, 4);
@@ -177,7 +184,7 @@ __device__ __forceinline__ void attention_decode_share(const DecodeParams& p, un
             }
         }
         if (i < my_tiles) {
-            const int tile = t0 + warp + i * WARPS;
+            const int tile = tile_at(t0 + warp + i * WARPS);
             const int key0 = tile * kTile;
             const int page = __shfl_sync(0xffffffffu, my_page, i % 32);
             const int64_t offset = page * p.page_stride + kv_head * p.head_stride +
@@ -310,7 +317,7 @@ __device__ __forceinline__ void attention_decode_share(const DecodeParams& p, un
         cp_async_wait<STAGES - 2>();
         __syncwarp();
         const unsigned char* stage = ring + (i % STAGES) * kStageBytes;
-        const int key0 = (t0 + warp + i * WARPS) * kTile;
+        const int key0 = tile_at(t0 + warp + i * WARPS) * kTile;
         if (patch && i == my_tiles - 1) {
             // the token's own tile: its row as this warp made it, over what the copy brought
             unsigned char* tile = ring + (i % STAGES) * kStageBytes;
@@ -343,7 +350,7 @@ __device__ __forceinline__ void attention_decode_share(const DecodeParams& p, un
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
                 const int key = key0 + 8 * j + 2 * tig + (e & 1);
-                const bool ok = key >= first && key < ctx;
+                const bool ok = (key >= first || (EXTRAS && key < keep)) && key < ctx;
                 float scaled = EXTRAS ? pl_exponent_of_score(s[j][e], p.scale_log2, p.cap_log2, p.scale_over_cap)
                                       : s[j][e] * p.scale_log2;
                 if (EXTRAS && p.distance_bias != nullptr && ok) {
@@ -1058,10 +1065,12 @@ int run_attention_decode(bool allow_cluster, const void* q, int64_t q_row_stride
     p.distance_bias = nullptr;
     p.bias_rows = 0;
     p.distance_slopes = nullptr;
+    p.keep_first = 0;
     if (extras != nullptr) {
         p.distance_bias = extras->distance_bias;
         p.bias_rows = extras->bias_rows;
         p.distance_slopes = extras->distance_slopes;
+        p.keep_first = extras->keep_first > 0 && window > 0 ? extras->keep_first : 0;
         PL_REQUIRE(p.distance_bias == nullptr || p.bias_rows > 0, "attention_decode: a distance bias needs rows");
         PL_REQUIRE(items == nullptr && tile_max == nullptr,
                    "attention_decode: sinks, gates and split weights are not taken over a work list or with attention mass");

@@ -8,7 +8,7 @@
 // a masked probability never multiplies stale memory). S = Q K^T and O += P V are
 // m16n8k16 bf16 MMAs with fp32 accumulators; the softmax is online, fp32, base 2
 // with the scale folded into the exponent; P is rounded to bf16 for the second
-// product. A query at position p reads keys max(0, p - window + 1) .. p. Tiles are
+// product. A query at position p reads keys max(0, p - window + 1) .. p (and the request's kept first keys). Tiles are
 // listed by the host, heaviest first. The order in which a query's keys are added
 // depends only on its position, not on how the prompt was cut: every portion walks
 // key tiles from the same 64-aligned starts.
@@ -53,6 +53,7 @@ struct PrefillParams {
     int bias_rows;
     const float* distance_slopes;  // fp32 [n_heads] (nullptr: none), see PlAttentionExtras
     int n_heads;
+    int keep_first;  // the request's first keys that stay in reach besides the window's, see PlAttentionExtras
 };
 
 // EXTRAS: the build that takes sinks, gates, split weights, a bias by distance and one pool for keys and values; the
@@ -78,7 +79,9 @@ __global__ void __launch_bounds__(kThreads, 2) attention_prefill_kernel(const Pr
 
     const int last_key = pos0 + n_rows - 1;
     const int first_key = p.window > 0 ? max(0, pos0 - p.window + 1) : 0;
-    const int j0 = first_key / kBN, j1 = last_key / kBN;
+    const int keep = EXTRAS ? p.keep_first : 0;
+    const PlTileWalk walk(first_key, keep, kBN);
+    const int n_walk = walk.count(last_key, kBN);
 
     // Q tile -> shared memory (zero rows past the portion's end).
     for (int c = threadIdx.x; c < kBM * kChunks; c += kThreads) {
@@ -98,7 +101,7 @@ __global__ void __launch_bounds__(kThreads, 2) attention_prefill_kernel(const Pr
         for (int c = threadIdx.x; c < kBN * kChunks; c += kThreads) {
             const int r = c / kChunks, ch = c % kChunks;
             const int key = j * kBN + r;
-            bool valid = key <= last_key && key >= first_key;
+            bool valid = key <= last_key && (key >= first_key || key < keep);
             int64_t offset = 0;
             if (valid) {
                 const int page = table_row[key / p.page_size];
@@ -121,7 +124,7 @@ __global__ void __launch_bounds__(kThreads, 2) attention_prefill_kernel(const Pr
         cp_async_commit();
     };
 
-    issue(j0, 0);
+    issue(walk.tile(0), 0);
     cp_async_wait<1>();  // Q has landed (the first K/V tile may still be in flight)
     __syncthreads();
 
@@ -146,10 +149,11 @@ __global__ void __launch_bounds__(kThreads, 2) attention_prefill_kernel(const Pr
     const int first_hi = p.window > 0 ? pos_hi - p.window + 1 : 0;
     const int warp_last = pos0 + warp * 16 + 15;  // the largest position among the warp's rows
 
-    for (int j = j0; j <= j1; ++j) {
-        const int stage = (j - j0) & 1;
-        if (j < j1) {
-            issue(j + 1, stage ^ 1);
+    for (int w = 0; w < n_walk; ++w) {
+        const int j = walk.tile(w);
+        const int stage = w & 1;
+        if (w + 1 < n_walk) {
+            issue(walk.tile(w + 1), stage ^ 1);
             cp_async_wait<1>();
         } else {
             cp_async_wait<0>();
@@ -160,7 +164,7 @@ __global__ void __launch_bounds__(kThreads, 2) attention_prefill_kernel(const Pr
         const int key0 = j * kBN;
         // A warp whose rows all come before this tile (causal) or after it (window) has nothing to add.
         const bool warp_active = key0 <= warp_last &&
-            (p.window <= 0 || key0 + kBN - 1 >= pos0 + warp * 16 - p.window + 1);
+            (p.window <= 0 || key0 + kBN - 1 >= pos0 + warp * 16 - p.window + 1 || key0 < keep);
         if (warp_active) {
             float s[kBN / 8][4];
 #pragma unroll
@@ -208,8 +212,8 @@ __global__ void __launch_bounds__(kThreads, 2) attention_prefill_kernel(const Pr
 #pragma unroll
                     for (int e = 0; e < 2; ++e) {
                         const int key = key0 + 8 * n + 2 * tig + e;
-                        s[n][e] = (key <= pos_lo && key >= first_lo) ? exponent_of(s[n][e], key, pos_lo) : -INFINITY;
-                        s[n][2 + e] = (key <= pos_hi && key >= first_hi) ? exponent_of(s[n][2 + e], key, pos_hi) : -INFINITY;
+                        s[n][e] = (key <= pos_lo && (key >= first_lo || key < keep)) ? exponent_of(s[n][e], key, pos_lo) : -INFINITY;
+                        s[n][2 + e] = (key <= pos_hi && (key >= first_hi || key < keep)) ? exponent_of(s[n][2 + e], key, pos_hi) : -INFINITY;
                     }
                     tile_lo = fmaxf(tile_lo, fmaxf(s[n][0], s[n][1]));
                     tile_hi = fmaxf(tile_hi, fmaxf(s[n][2], s[n][3]));
@@ -336,7 +340,7 @@ int launch_prefill_build(const PrefillParams& p, int n_tiles, int n_heads, cudaS
 template <int HD>
 int launch_prefill(const PrefillParams& p, int n_tiles, int n_heads, cudaStream_t stream) {
     const bool extras = p.sinks != nullptr || p.gate != nullptr || p.split_weights || p.v_pool == p.k_pool ||
-                        p.cap_log2 > 0.0f || p.distance_bias != nullptr || p.distance_slopes != nullptr;
+                        p.cap_log2 > 0.0f || p.distance_bias != nullptr || p.distance_slopes != nullptr || p.keep_first > 0;
     return extras ? launch_prefill_build<HD, true>(p, n_tiles, n_heads, stream)
                   : launch_prefill_build<HD, false>(p, n_tiles, n_heads, stream);
 }
@@ -401,6 +405,7 @@ PL_API int pl_attention_prefill(const void* q, int64_t q_row_stride, const void*
     p.bias_rows = extras != nullptr ? extras->bias_rows : 0;
     p.distance_slopes = extras != nullptr ? extras->distance_slopes : nullptr;
     p.n_heads = n_heads;
+    p.keep_first = extras != nullptr && extras->keep_first > 0 ? extras->keep_first : 0;
     PL_REQUIRE(p.distance_bias == nullptr || p.bias_rows > 0, "attention_prefill: a distance bias needs rows");
     p.cap_log2 = p.scale_over_cap = 0.0f;
     if (extras != nullptr && extras->softcap > 0.0f) {

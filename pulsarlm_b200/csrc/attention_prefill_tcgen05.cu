@@ -87,10 +87,13 @@ struct TcPrefillParams {
     // score; and a sink per head, exp(sinks[h]) in the row's denominator (nullptr: none).
     const float* slopes;
     const float* sinks;
+    // (the builds with kReach only) the request's first keys that stay in reach besides the window's
+    int keep_first;
 };
 
-// What a build adds to its scores by distance.
-enum BiasKind : int { kBiasNone = 0, kBiasTable = 1, kBiasSlopes = 2 };
+// What a build adds to its scores by distance; kReach adds nothing to the scores but takes a sink per head and kept
+// first keys.
+enum BiasKind : int { kBiasNone = 0, kBiasTable = 1, kBiasSlopes = 2, kReach = 3 };
 
 // What pl_attention_prefill_tcgen05 needs to measure attention mass: the rows' weights,
 // zeroed scratch of n_tiles * n_heads * 8 * pages floats (pages >= the block table's
@@ -201,10 +204,14 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
     const int last_key = pos0 + n_rows - 1;
     const int first_key = p.window > 0 ? max(0, pos0 - p.window + 1) : 0;
     // This CTA's share of the tile's 64-key tiles (all of them without splits).
-    const int all_tiles = last_key / kKeys - first_key / kKeys + 1;
+    // (kReach: the walk jumps from the kept first keys' tiles to the window's)
+    const int keep = BIAS == kReach ? p.keep_first : 0;
+    const PlTileWalk walk(first_key, keep, kKeys);
+    const int all_tiles = walk.count(last_key, kKeys);
     const int per_split = (all_tiles + p.n_splits - 1) / p.n_splits;
     const int j_begin = min(all_tiles, static_cast<int>(blockIdx.z) * per_split);
     const int j0 = first_key / kKeys + j_begin, n_tiles = min(all_tiles, j_begin + per_split) - j_begin;
+    auto tile_of = [&](int j) { return BIAS == kReach ? walk.tile(j_begin + j) : j0 + j; };  // the j-th tile of this share
     if (n_tiles == 0) {
         // Nothing for this split: its rows say so (the merge skips a split whose base is -inf).
         for (int i = threadIdx.x; i < HEADS * kRows; i += kThreadsTc) {
@@ -267,8 +274,20 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
             if (j % (32 / kPieces) == 0) {
                 // Pieces outside [first_key, last_key] are never attended (masked): they
                 // are filled from the nearest needed piece, whose page is held.
-                my_key = (j0 + j) * kKeys + lane * kPiece;
-                my_key = min(max(my_key, (first_key / kPiece) * kPiece), (last_key / kPiece) * kPiece);
+                if constexpr (BIAS == kReach) {
+                    my_key = tile_of(j + lane / kPieces) * kKeys + (lane % kPieces) * kPiece;
+                    // (a piece between the kept keys and the window is never attended: in a kept keys' tile the last
+                    // kept piece stands in for it, else the window's first)
+                    if (j_begin + j + lane / kPieces < walk.head) {
+                        my_key = min(my_key, (keep - 1) / kPiece * kPiece);
+                    } else if (my_key >= keep) {
+                        my_key = max(my_key, (first_key / kPiece) * kPiece);
+                    }
+                    my_key = min(my_key, (last_key / kPiece) * kPiece);
+                } else {
+                    my_key = (j0 + j) * kKeys + lane * kPiece;
+                    my_key = min(max(my_key, (first_key / kPiece) * kPiece), (last_key / kPiece) * kPiece);
+                }
                 my_page = table_row[my_key / p.page_size];
                 if (my_page < 0 || my_page >= p.n_pages) {
                     if (my_key <= (last_key / kPiece) * kPiece && p.status != nullptr) {
@@ -517,7 +536,8 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
             if (!kTurns && lane == 0) {
                 mbar_arrive(&s_free[hs][b]);
             }
-            const int key0 = (j0 + j) * kKeys + part * kMyKeys;
+            const int tile_key = tile_of(j) * kKeys;
+            const int key0 = tile_key + part * kMyKeys;
             if constexpr (BIAS == kBiasTable) {
                 // this row's bias at every key's distance (neighbouring keys, neighbouring entries of the head's row)
                 const float* bias_row = p.bias + static_cast<int64_t>(head) * p.bias_rows;
@@ -542,15 +562,14 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
                     s[c + 1] = biased.y;
                 }
             }
-            const bool edge = (j0 + j) * kKeys + kKeys - 1 > pos0 ||
-                (p.window > 0 && (j0 + j) * kKeys < pos0 + kSpan - p.window);
+            const bool edge = tile_key + kKeys - 1 > pos0 || (p.window > 0 && tile_key < pos0 + kSpan - p.window);
             // The tile's maximum, on the raw products (the scale is positive), four running
             // maxima side by side so that the chain of dependent instructions stays short.
             if (edge) {
 #pragma unroll
                 for (int c = 0; c < kMyKeys; ++c) {
                     const int key = key0 + c;
-                    s[c] = (key <= pos && key >= first) ? s[c] : -INFINITY;
+                    s[c] = (key <= pos && (key >= first || (BIAS == kReach && key < keep))) ? s[c] : -INFINITY;
                 }
             }
             if constexpr (kMyKeys == kKeys) {
@@ -705,7 +724,7 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
                 }
             }
         } else if (ok) {
-            const float inv = BIAS == kBiasSlopes ? pl_attention_row_factor(m, l, p.sinks, nullptr, 0, 0, head)
+            const float inv = BIAS == kBiasSlopes || BIAS == kReach ? pl_attention_row_factor(m, l, p.sinks, nullptr, 0, 0, head)
                                                   : (l > 0.0f ? 1.0f / l : 0.0f);
             __nv_bfloat16* dst = p.out + (row0 + rr) * p.out_row_stride + static_cast<int64_t>(head) * HD +
                 part * kMyDims;
@@ -921,7 +940,7 @@ static int run_tc_prefill(const void* q, int64_t q_row_stride, int n_tokens, con
                           int n_tiles, void* out, int64_t out_row_stride, int n_heads, int n_kv_heads,
                           int head_dim, int window, float scale, int n_splits, float* scratch,
                           int wide, const PlPrefillMass* mass, const float* bias, int bias_rows, const float* slopes,
-                          const float* sinks, int32_t* status, cudaStream_t stream) {
+                          const float* sinks, int keep_first, int32_t* status, cudaStream_t stream) {
     PL_REQUIRE(n_tiles >= 0 && n_heads > 0 && n_kv_heads > 0 && n_heads % n_kv_heads == 0 && n_tokens > 0,
                "attention_prefill_tcgen05: bad sizes tiles=%d heads=%d kv_heads=%d tokens=%d", n_tiles, n_heads,
                n_kv_heads, n_tokens);
@@ -988,8 +1007,11 @@ static int run_tc_prefill(const void* q, int64_t q_row_stride, int n_tokens, con
     p.inv_scale = 1.0f / scale;
     p.slopes = slopes;
     p.sinks = sinks;
-    PL_REQUIRE(slopes == nullptr ? sinks == nullptr : bias == nullptr && mass == nullptr,
-               "attention_prefill_tcgen05: a linear bias is taken without a table and without attention mass, a sink only with it");
+    p.keep_first = window > 0 && keep_first > 0 ? keep_first : 0;
+    PL_REQUIRE((slopes == nullptr && sinks == nullptr && p.keep_first == 0) || (bias == nullptr && mass == nullptr),
+               "attention_prefill_tcgen05: a linear bias, sinks and kept first keys are taken without a table and without attention mass");
+    PL_REQUIRE(slopes == nullptr || p.keep_first == 0, "attention_prefill_tcgen05: kept first keys are not taken with a linear bias");
+    const bool reach = slopes == nullptr && (sinks != nullptr || p.keep_first > 0);
     if (bias != nullptr) {
         PL_REQUIRE(pairs && mass == nullptr && bias_rows > 0,
                    "attention_prefill_tcgen05: a bias by distance is taken with two heads of a kv head per CTA (an even "
@@ -1026,6 +1048,12 @@ static int run_tc_prefill(const void* q, int64_t q_row_stride, int n_tokens, con
     } else if (slopes != nullptr) {
         code = pairs ? launch_tc_prefill<128, 2, false, kBiasSlopes>(mq, mk, mv, p, n_tiles, n_heads, stream)
                      : launch_tc_prefill<128, 2, true, kBiasSlopes>(mq, mk, mv, p, n_tiles, n_heads, stream);
+    } else if (reach && head_dim == 64) {
+        code = pairs ? launch_tc_prefill<64, 2, false, kReach>(mq, mk, mv, p, n_tiles, n_heads, stream)
+                     : launch_tc_prefill<64, 2, true, kReach>(mq, mk, mv, p, n_tiles, n_heads, stream);
+    } else if (reach) {
+        code = pairs ? launch_tc_prefill<128, 2, false, kReach>(mq, mk, mv, p, n_tiles, n_heads, stream)
+                     : launch_tc_prefill<128, 2, true, kReach>(mq, mk, mv, p, n_tiles, n_heads, stream);
     } else if (head_dim == 64) {
         code = pairs ? launch_tc_prefill<64, 2, false>(mq, mk, mv, p, n_tiles, n_heads, stream)
             : wide   ? launch_tc_prefill<64, 2, true>(mq, mk, mv, p, n_tiles, n_heads, stream)
@@ -1055,7 +1083,7 @@ PL_API int pl_attention_prefill_tcgen05(const void* q, int64_t q_row_stride, int
                                         int wide, const PlPrefillMass* mass, int32_t* status, cudaStream_t stream) {
     return run_tc_prefill(q, q_row_stride, n_tokens, k_pool, v_pool, page_stride, head_stride, page_size, n_pages, table,
                           table_width, tiles, n_tiles, out, out_row_stride, n_heads, n_kv_heads, head_dim, window, scale,
-                          n_splits, scratch, wide, mass, nullptr, 0, nullptr, nullptr, status, stream);
+                          n_splits, scratch, wide, mass, nullptr, 0, nullptr, nullptr, 0, status, stream);
 }
 
 // The same with a bias by distance: bias fp32 [n_heads, bias_rows] (a head's entries side by side);
@@ -1071,7 +1099,7 @@ PL_API int pl_attention_prefill_tcgen05_bias(const void* q, int64_t q_row_stride
     PL_REQUIRE(bias != nullptr && bias_rows > 0, "attention_prefill_tcgen05_bias: needs a bias table");
     return run_tc_prefill(q, q_row_stride, n_tokens, k_pool, v_pool, page_stride, head_stride, page_size, n_pages, table,
                           table_width, tiles, n_tiles, out, out_row_stride, n_heads, n_kv_heads, head_dim, window, scale,
-                          n_splits, scratch, 0, nullptr, bias, bias_rows, nullptr, nullptr, status, stream);
+                          n_splits, scratch, 0, nullptr, bias, bias_rows, nullptr, nullptr, 0, status, stream);
 }
 
 // The same with a linear bias and, optionally, a sink: slopes fp32 [n_heads], slopes[h] * d is taken off head h's
@@ -1087,5 +1115,22 @@ PL_API int pl_attention_prefill_tcgen05_slopes(const void* q, int64_t q_row_stri
     PL_REQUIRE(slopes != nullptr, "attention_prefill_tcgen05_slopes: needs the heads' slopes");
     return run_tc_prefill(q, q_row_stride, n_tokens, k_pool, v_pool, page_stride, head_stride, page_size, n_pages, table,
                           table_width, tiles, n_tiles, out, out_row_stride, n_heads, n_kv_heads, head_dim, window, scale,
-                          n_splits, scratch, n_heads / n_kv_heads % 2, nullptr, nullptr, 0, slopes, sinks, status, stream);
+                          n_splits, scratch, n_heads / n_kv_heads % 2, nullptr, nullptr, 0, slopes, sinks, 0, status, stream);
+}
+
+// The same with a sink per head and kept first keys, nothing by distance: sinks fp32 [n_heads] (may be nullptr),
+// exp(sinks[h]) joins head h's denominator; keep_first >= 0, the request's first keys that stay in reach besides the
+// window's. Any GQA group (an odd one takes tiles of up to 256 rows); no attention mass.
+PL_API int pl_attention_prefill_tcgen05_reach(const void* q, int64_t q_row_stride, int n_tokens, const void* k_pool,
+                                              const void* v_pool, int64_t page_stride, int64_t head_stride,
+                                              int page_size, int n_pages, const int32_t* table, int table_width,
+                                              const int32_t* tiles, int n_tiles, void* out, int64_t out_row_stride,
+                                              int n_heads, int n_kv_heads, int head_dim, int window, float scale,
+                                              int n_splits, float* scratch, const float* sinks, int keep_first,
+                                              int32_t* status, cudaStream_t stream) {
+    PL_REQUIRE(sinks != nullptr || keep_first > 0, "attention_prefill_tcgen05_reach: needs sinks or kept first keys");
+    return run_tc_prefill(q, q_row_stride, n_tokens, k_pool, v_pool, page_stride, head_stride, page_size, n_pages, table,
+                          table_width, tiles, n_tiles, out, out_row_stride, n_heads, n_kv_heads, head_dim, window, scale,
+                          n_splits, scratch, n_heads / n_kv_heads % 2, nullptr, nullptr, 0, nullptr, sinks, keep_first,
+                          status, stream);
 }

@@ -77,13 +77,15 @@ __global__ void attention_simt_kernel(const scalar_t* __restrict__ q, int64_t q_
                                       const float* __restrict__ query_weights, const float* __restrict__ sinks,
                                       const scalar_t* __restrict__ gate, int64_t gate_row_stride,
                                       const float* __restrict__ distance_bias, int bias_rows,
-                                      const float* __restrict__ distance_slopes, int32_t* status) {
+                                      const float* __restrict__ distance_slopes, int keep_first, int32_t* status) {
     extern __shared__ float q_shared[];  // [warps][head_dim]
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
     const int t = blockIdx.x;
     const int kv_head = blockIdx.y;
     const int p = pos[t];
     const int first = window > 0 ? max(0, p - window + 1) : 0;
+    const PlTileWalk walk(first, keep_first, 32);
+    const int chunks = walk.count(p, 32);
     const int32_t* row = table + static_cast<int64_t>(entry[t]) * table_width;
     float* qs = q_shared + warp * head_dim;
     const int n_acc = (head_dim + 31) / 32;
@@ -121,9 +123,10 @@ __global__ void attention_simt_kernel(const scalar_t* __restrict__ q, int64_t q_
             }
         };
 
-        for (int base = (first / 32) * 32; base <= p; base += 32) {
+        for (int w = 0; w < chunks; ++w) {
+            const int base = walk.tile(w) * 32;
             const int j = base + lane;
-            const bool valid = j >= first && j <= p;
+            const bool valid = (j >= first || j < keep_first) && j <= p;
             int64_t offset = -1;
             float s = -INFINITY;
             if (valid) {
@@ -150,7 +153,7 @@ __global__ void attention_simt_kernel(const scalar_t* __restrict__ q, int64_t q_
                 // Largest scaled score per page; a page may span several chunks, so the
                 // running maximum is flushed only when the walk leaves the page.
                 const int last = min(base + 31, p);
-                for (int pg = max(base, first) / page_size; pg <= last / page_size; ++pg) {
+                for (int pg = (base < keep_first ? base : max(base, first)) / page_size; pg <= last / page_size; ++pg) {
                     const float chunk_max = pl_warp_max(valid && j / page_size == pg ? s : -INFINITY);
                     if (pg != mass_page) {
                         add_mass(mass_page, mass_max);
@@ -240,7 +243,8 @@ __global__ void attention_simt_kernel(const scalar_t* __restrict__ q, int64_t q_
 // h's output for token t is multiplied by sigmoid(gate[t, h]). distance_bias (fp32 [n_heads,
 // bias_rows], may be nullptr): distance_bias[h, min(pos - key's position, bias_rows - 1)] is added
 // to head h's scaled score. distance_slopes (fp32 [n_heads], may be nullptr): distance_slopes[h] times the
-// distance is taken off head h's scaled score.
+// distance is taken off head h's scaled score. keep_first > 0: the request's first keep_first keys stay in reach
+// besides the window's.
 PL_API int pl_attention_simt(const void* q, int64_t q_row_stride, const void* k_pool, const void* v_pool,
                              int64_t page_stride, int64_t head_stride, int page_size, int n_pages,
                              const int32_t* table, int table_width, const int32_t* pos, const int32_t* entry,
@@ -248,7 +252,7 @@ PL_API int pl_attention_simt(const void* q, int64_t q_row_stride, const void* k_
                              int head_dim, int window, float scale, float softcap, int dtype, float* mass_sum,
                              float* weight_sum, const float* query_weights, const float* sinks, const void* gate,
                              int64_t gate_row_stride, const float* distance_bias, int bias_rows,
-                             const float* distance_slopes, int32_t* status, cudaStream_t stream) {
+                             const float* distance_slopes, int keep_first, int32_t* status, cudaStream_t stream) {
     PL_REQUIRE(n_tokens >= 0 && n_heads > 0 && n_kv_heads > 0 && head_dim > 0 && page_size > 0,
                "attention: bad sizes tokens=%d heads=%d kv_heads=%d head_dim=%d page=%d", n_tokens, n_heads,
                n_kv_heads, head_dim, page_size);
@@ -275,7 +279,7 @@ PL_API int pl_attention_simt(const void* q, int64_t q_row_stride, const void* k_
             static_cast<const scalar_t*>(v_pool), page_stride, head_stride, page_size, n_pages, table, table_width,
             pos, entry, static_cast<scalar_t*>(out), out_row_stride, n_heads, group, head_dim, window, scale,
             softcap, mass_sum, weight_sum, query_weights, sinks, static_cast<const scalar_t*>(gate), gate_row_stride,
-            distance_bias, bias_rows, distance_slopes, status);
+            distance_bias, bias_rows, distance_slopes, keep_first > 0 ? keep_first : 0, status);
     });
     PL_CHECK_LAUNCH("attention");
     return 0;

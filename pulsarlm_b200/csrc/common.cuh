@@ -162,7 +162,8 @@ __device__ __forceinline__ float pl_block_max(float v, float* scratch) {
 // (a head's entries side by side); distance_bias[h, min(d, bias_rows - 1)] joins head h's scaled (and
 // capped) score of a key d tokens before the query; the scale does not touch it. distance_slopes: fp32
 // [n_heads]; distance_slopes[h] * d is taken off head h's scaled (and capped) score of a key d tokens
-// before the query, for any d (a linear bias without a table's end).
+// before the query, for any d (a linear bias without a table's end). keep_first: with a window, the sequence's
+// first keep_first keys stay in reach of every query after them besides the window's.
 struct PlAttentionExtras {
     const float* sinks;
     const void* gate;
@@ -172,6 +173,20 @@ struct PlAttentionExtras {
     const float* distance_bias;
     int bias_rows;
     const float* distance_slopes;
+    int keep_first;
+};
+
+// The tiles of `size` keys that a walk from key `first` (a window's first key) to the last key takes when the
+// sequence's first `keep` keys stay in reach: tiles 0 .. head - 1 hold kept keys, tile `start` the window's first,
+// and place w of the walk is tile w below head, else start + w - head. (Kept keys that reach the window's first
+// tile: head == start, one run from tile 0 on.)
+struct PlTileWalk {
+    int head, start;
+    __device__ __forceinline__ PlTileWalk(int first, int keep, int size)
+    : head(min((keep + size - 1) / size, first / size)), start(first / size) {}
+    __device__ __forceinline__ int tile(int w) const { return w < head ? w : start + w - head; }
+    // Places from the first to the tile of key `last`.
+    __device__ __forceinline__ int count(int last, int size) const { return head + last / size - start + 1; }
 };
 
 // A raw score on its way into the base-2 softmax: times scale * log2 e, or with a cap

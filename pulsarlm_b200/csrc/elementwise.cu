@@ -4,6 +4,7 @@
 // never rounded to bfloat16. Norm statistics, the SiLU and the products are fp32
 // with one rounding on store.
 #include "common.cuh"
+#include "gate_units.cuh"
 
 #include <algorithm>
 
@@ -392,7 +393,7 @@ PL_API int pl_fill_random(void* out, int64_t n, int dtype, uint64_t seed, uint64
 
 // ---------------------------------------------------------------------------
 // Bias and activation of a plain projection: out = act(in + bias), fp32 inside.
-// act 0: none, 1: relu(z)^2, 2: tanh(z). Rows of `in` may be columns of a wider
+// act 0: none, 1: relu(z)^2, 2: tanh(z), 3: gelu(z). Rows of `in` may be columns of a wider
 // matrix (in_row_stride elements apart); out is dense and may be `in` itself.
 namespace {
 
@@ -410,12 +411,7 @@ __global__ void bias_act_kernel(const scalar_t* in, int64_t in_row_stride, const
         if (bias != nullptr) {
             z += pl_load(bias + c);
         }
-        if (act == 1) {
-            z = z > 0.0f ? z * z : 0.0f;
-        } else if (act == 2) {
-            z = tanhf(z);
-        }
-        pl_store(out + i, z);
+        pl_store(out + i, pl_plain_activation(z, act));
     }
 }
 
@@ -436,14 +432,8 @@ __global__ void bias_act_vec_kernel(const scalar_t* in, int64_t in_row_stride, c
             const float4 b = pl_load4(bias + c);
             z.x += b.x; z.y += b.y; z.z += b.z; z.w += b.w;
         }
-        if (act == 1) {
-            z.x = z.x > 0.0f ? z.x * z.x : 0.0f;
-            z.y = z.y > 0.0f ? z.y * z.y : 0.0f;
-            z.z = z.z > 0.0f ? z.z * z.z : 0.0f;
-            z.w = z.w > 0.0f ? z.w * z.w : 0.0f;
-        } else if (act == 2) {
-            z = make_float4(tanhf(z.x), tanhf(z.y), tanhf(z.z), tanhf(z.w));
-        }
+        z = make_float4(pl_plain_activation(z.x, act), pl_plain_activation(z.y, act), pl_plain_activation(z.z, act),
+                        pl_plain_activation(z.w, act));
         pl_store4(out + t * width + c, z);
     }
 }
@@ -452,7 +442,7 @@ __global__ void bias_act_vec_kernel(const scalar_t* in, int64_t in_row_stride, c
 
 PL_API int pl_bias_act(const void* in, int64_t in_row_stride, const void* bias, void* out, int n_tokens, int width,
                        int act, int dtype, cudaStream_t stream) {
-    PL_REQUIRE(n_tokens >= 0 && width > 0 && act >= 0 && act <= 2 && in_row_stride >= width,
+    PL_REQUIRE(n_tokens >= 0 && width > 0 && act >= 0 && act <= 3 && in_row_stride >= width,
                "bias_act: bad arguments tokens=%d width=%d act=%d", n_tokens, width, act);
     if (n_tokens == 0) {
         return 0;

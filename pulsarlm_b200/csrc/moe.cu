@@ -1,7 +1,7 @@
 // A routed feed-forward (mixture of experts): the router, and the experts' products for
 // steps of few tokens and for the float32 engine.
 //
-// Router (pl_moe_route), all fp32: logits z = W_r h, scores s = softmax(z) over all experts
+// Router (pl_moe_route), all fp32: logits z = W_r h (+ a bias per expert, `logit_bias`), scores s = softmax(z) over all experts
 // (or, `sigmoid_scores`, s = sigmoid(z) of each alone), choice scores c = s + correction.
 // Experts form `n_groups` equal groups of neighbours; a group's score is the sum of its
 // `group_top` largest choice scores (1: its largest), and only experts of the `keep` best
@@ -12,7 +12,7 @@
 //
 // Experts (pl_moe_gate_up, pl_moe_down): expert e of a token computes W_down,e (silu(W_gate,e h)
 // * (W_up,e h)); pl_moe_up takes the place of pl_moe_gate_up for experts without a gate, W_down,e
-// act(W_up,e h) with act the square of relu. With `clamped` the unit is gate_units.cuh's, and a pair's weight, where
+// act(W_up,e h) with act the square of relu or the exact GELU. With `clamped` the unit is gate_units.cuh's, and a pair's weight, where
 // given, multiplies the expert's input (its gate and up products: a linear map carries the weight through) instead of
 // its output. The first kernel takes a (token, chosen expert) pair per block row and writes
 // the gated activation, a warp per feature (both rows of the feature read with 16-byte loads,
@@ -77,7 +77,8 @@ struct Vec<__nv_bfloat16> {
 // chooses. A token's sums are the same whatever TOKENS is.
 template <typename scalar_t, int TOKENS>
 __global__ void __launch_bounds__(512, TOKENS > 1 ? 2 : 1) moe_route_kernel(const scalar_t* __restrict__ h, int64_t h_stride, const float* __restrict__ router,
-                                 const float* __restrict__ correction, int32_t* __restrict__ ids,
+                                 const float* __restrict__ logit_bias, const float* __restrict__ correction,
+                                 int32_t* __restrict__ ids,
                                  float* __restrict__ weights, int n_tokens, int hidden, int n_experts, int top,
                                  int n_groups, int keep, int sigmoid_scores, int group_top, int renormalise,
                                  float* __restrict__ shared_weights) {
@@ -166,7 +167,7 @@ __global__ void __launch_bounds__(512, TOKENS > 1 ? 2 : 1) moe_route_kernel(cons
         for (int r = 0; r < TOKENS; ++r) {
             const float total = pl_warp_sum(z[r]);
             if (lane == 0) {
-                scores[r * n_rows + e] = total;
+                scores[r * n_rows + e] = logit_bias != nullptr && e < n_experts ? total + logit_bias[e] : total;
             }
         }
     }
@@ -448,11 +449,11 @@ __global__ void moe_gate_up_kernel(const scalar_t* __restrict__ h, int64_t h_str
     }
 }
 
-// Block (pair, feature block): act[pair, f] = relu(up_e[f] . h)^2, for experts without a gate.
+// Block (pair, feature block): act[pair, f] = a(up_e[f] . h), for experts without a gate (a by pl_plain_activation's code).
 template <typename scalar_t>
 __global__ void moe_up_kernel(const scalar_t* __restrict__ h, int64_t h_stride, const scalar_t* __restrict__ up,
                               const int32_t* __restrict__ ids, scalar_t* __restrict__ act, int hidden, int ff, int top,
-                              int n_experts, int vectors) {
+                              int n_experts, int vectors, int activation) {
     pl_grid_trigger();
     pl_grid_wait();
     extern __shared__ float row[];  // [hidden]
@@ -479,16 +480,14 @@ __global__ void moe_up_kernel(const scalar_t* __restrict__ h, int64_t h_stride, 
             for (int r = 1; r < kFeaturesPerWarp; ++r) {
                 ul = lane == r ? u[r] : ul;
             }
-            ul = fmaxf(ul, 0.0f);
-            pl_store(act + static_cast<int64_t>(pair) * ff + f0 + lane, ul * ul);
+            pl_store(act + static_cast<int64_t>(pair) * ff + f0 + lane, pl_plain_activation(ul, activation));
         }
         return;
     }
     for (int f = f0; f < min(f0 + kFeaturesPerWarp, ff); ++f) {
-        float u = warp_dot<scalar_t>(weights + static_cast<int64_t>(f) * hidden, row, hidden, vectors, lane);
+        const float u = warp_dot<scalar_t>(weights + static_cast<int64_t>(f) * hidden, row, hidden, vectors, lane);
         if (lane == 0) {
-            u = fmaxf(u, 0.0f);
-            pl_store(act + static_cast<int64_t>(pair) * ff + f, u * u);
+            pl_store(act + static_cast<int64_t>(pair) * ff + f, pl_plain_activation(u, activation));
         }
     }
 }
@@ -706,7 +705,8 @@ __global__ void moe_combine_kernel(const scalar_t* __restrict__ y, const int32_t
 // sigmoid_scores: s = sigmoid(z) instead of softmax(z); group_top: how many of a group's largest choice
 // scores add up to its score; renormalise: whether the chosen scores are divided by their sum. shared_weights (fp32
 // [T], may be nullptr): sigmoid of the logit of one more row of the router, a shared expert's gate.
-PL_API int pl_moe_route(const void* h, int64_t h_stride, const float* router, const float* correction, int32_t* ids,
+PL_API int pl_moe_route(const void* h, int64_t h_stride, const float* router, const float* logit_bias,
+                        const float* correction, int32_t* ids,
                         float* weights, int n_tokens, int hidden, int n_experts, int top, int n_groups, int keep,
                         int sigmoid_scores, int group_top, int renormalise, float* shared_weights, int dtype,
                         cudaStream_t stream) {
@@ -740,7 +740,7 @@ PL_API int pl_moe_route(const void* h, int64_t h_stride, const float* router, co
             // (room for two of these CTAs' rows per SM)
             cudaFuncSetAttribute(moe_route_kernel<scalar_t, 8>, cudaFuncAttributePreferredSharedMemoryCarveout, 100);
             pl_launch_overlapped(moe_route_kernel<scalar_t, 8>, dim3((n_tokens + 7) / 8), dim3(threads), smem, stream,
-                                 static_cast<const scalar_t*>(h), h_stride, router, correction, ids, weights, n_tokens,
+                                 static_cast<const scalar_t*>(h), h_stride, router, logit_bias, correction, ids, weights, n_tokens,
                                  hidden, n_experts, top, n_groups, keep, sigmoid_scores, group_top, renormalise,
                                  shared_weights);
         } else {
@@ -749,7 +749,7 @@ PL_API int pl_moe_route(const void* h, int64_t h_stride, const float* router, co
                                      static_cast<int>(smem));
             }
             pl_launch_overlapped(moe_route_kernel<scalar_t, 1>, dim3(n_tokens), dim3(threads), smem, stream,
-                                 static_cast<const scalar_t*>(h), h_stride, router, correction, ids, weights, n_tokens,
+                                 static_cast<const scalar_t*>(h), h_stride, router, logit_bias, correction, ids, weights, n_tokens,
                                  hidden, n_experts, top, n_groups, keep, sigmoid_scores, group_top, renormalise,
                                  shared_weights);
         }
@@ -788,10 +788,12 @@ PL_API int pl_moe_gate_up(const void* h, int64_t h_stride, const void* gate_up, 
     return 0;
 }
 
-// up [n_experts, ff, hidden]; act [T * top, ff] = relu(up_e h)^2 for each pair's expert e.
+// up [n_experts, ff, hidden]; act [T * top, ff] = a(up_e h) for each pair's expert e; activation 1: the square of relu,
+// 3: the exact GELU (pl_plain_activation).
 PL_API int pl_moe_up(const void* h, int64_t h_stride, const void* up, const int32_t* ids, void* act, int n_tokens,
-                     int hidden, int ff, int top, int n_experts, int dtype, cudaStream_t stream) {
+                     int hidden, int ff, int top, int n_experts, int activation, int dtype, cudaStream_t stream) {
     PL_REQUIRE(n_tokens >= 0 && hidden > 0 && ff > 0 && top > 0 && n_experts > 0, "moe_up: bad sizes");
+    PL_REQUIRE(activation == 1 || activation == 3, "moe_up: unknown activation %d", activation);
     const size_t smem = static_cast<size_t>(hidden) * sizeof(float);
     PL_REQUIRE(smem <= 200 * 1024, "moe_up: hidden %d is too wide", hidden);
     if (n_tokens == 0) {
@@ -808,7 +810,7 @@ PL_API int pl_moe_up(const void* h, int64_t h_stride, const void* up, const int3
         }
         pl_launch_overlapped(moe_up_kernel<scalar_t>, grid, dim3(warps * 32), smem, stream,
                              static_cast<const scalar_t*>(h), h_stride, static_cast<const scalar_t*>(up), ids,
-                             static_cast<scalar_t*>(act), hidden, ff, top, n_experts, vectors);
+                             static_cast<scalar_t*>(act), hidden, ff, top, n_experts, vectors, activation);
     });
     PL_CHECK_LAUNCH("moe_up");
     return 0;

@@ -42,11 +42,13 @@ bool PagePool::give(const int* pages, int count) {
 
 // ------------------------------------------------------------------ CacheBook
 
-CacheBook::CacheBook(int n_groups, const int* windows, int page_size, const int* n_pages, int max_requests,
-                     bool track_fresh)
+CacheBook::CacheBook(int n_groups, const int* windows, const int* keep_first, int page_size, const int* n_pages,
+                     int max_requests, bool track_fresh)
 : page_size_(page_size), max_requests_(max_requests), track_fresh_(track_fresh) {
     for (int g = 0; g < n_groups; ++g) {
         windows_.push_back(windows != nullptr ? windows[g] : -1);
+        const int kept = keep_first != nullptr && keep_first[g] > 0 ? keep_first[g] : 0;
+        kept_pages_.push_back((kept + page_size - 1) / page_size);
         pools_.emplace_back(n_pages[g]);  // (a group whose window lets pages go needs fewer than one that keeps all)
         fresh_.emplace_back();
     }
@@ -148,7 +150,7 @@ int CacheBook::commit(int64_t request, int64_t new_len) {
     for (size_t g = 0; g < pools_.size(); ++g) {
         std::vector<int>& pages = r.pages[g];
         const int first = std::min<int>(first_needed_page(static_cast<int>(g), new_len), static_cast<int>(pages.size()));
-        for (int i = 0; i < first; ++i) {
+        for (int i = kept_pages_[g]; i < first; ++i) {
             if (pages[i] >= 0) {
                 if (!pools_[g].give(&pages[i], 1)) {
                     return kBadPage;
@@ -494,9 +496,10 @@ PLH_API int plh_pool_stat(void* pool, int what) {
 }
 PLH_API int plh_pool_is_held(void* pool, int page) { return static_cast<PagePool*>(pool)->is_held(page) ? 1 : 0; }
 
-PLH_API void* plh_cache_create(int n_groups, const int32_t* windows, int page_size, const int32_t* n_pages,
+PLH_API void* plh_cache_create(int n_groups, const int32_t* windows, const int32_t* keep_first, int page_size,
+                               const int32_t* n_pages,
                                int max_requests, int track_fresh) {
-    return new CacheBook(n_groups, windows, page_size, n_pages, max_requests, track_fresh != 0);
+    return new CacheBook(n_groups, windows, keep_first, page_size, n_pages, max_requests, track_fresh != 0);
 }
 PLH_API void plh_cache_destroy(void* cache) { delete static_cast<CacheBook*>(cache); }
 PLH_API int plh_cache_open(void* cache, int64_t request) { return static_cast<CacheBook*>(cache)->open(request); }

@@ -52,10 +52,12 @@ enum Code : int {
 
 // Bookkeeping of the cache manager: per group a pool (and an optional window), per
 // request a slot, a length and one page list per group (-1 where a windowed group
-// gave the page back).
+// gave the page back). A windowed group may keep a sequence's first tokens in reach
+// besides the window: the pages that hold them are never given back before the end.
 class CacheBook {
 public:
-    CacheBook(int n_groups, const int* windows, int page_size, const int* n_pages, int max_requests, bool track_fresh);
+    CacheBook(int n_groups, const int* windows, const int* keep_first, int page_size, const int* n_pages, int max_requests,
+              bool track_fresh);
 
     int open(int64_t request);  // slot, kNoRoom as -100, or kAlreadyOpen
     bool is_open(int64_t request) const { return requests_.count(request) != 0; }
@@ -91,6 +93,7 @@ private:
     int max_requests_;
     bool track_fresh_;
     std::vector<int> windows_;
+    std::vector<int> kept_pages_;  // leading pages of a request that a windowed group keeps
     std::vector<PagePool> pools_;
     std::vector<int> free_slots_;
     std::unordered_map<int64_t, Request> requests_;

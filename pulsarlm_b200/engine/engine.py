@@ -145,6 +145,13 @@ class Engine:
         bad = [t for t in tokens if not 0 <= t < self.vocab_size]
         if bad:
             raise ValueError(f"token id {bad[0]} is outside [0, {self.vocab_size})")
+        limit = self.model.spec.max_positions
+        if limit is not None:
+            # (a model with a table of positions: the last token drawn needs no position of its own)
+            if len(tokens) > limit:
+                raise ValueError(f"a request of {len(tokens)} tokens exceeds the model's {limit} positions")
+            room = limit - len(tokens) + 1
+            max_tokens = room if max_tokens is None else min(max_tokens, room)
         sampling = sampling or SamplingParams()
         request = Request(next(self._ids), tokens, sampling, max_tokens, ignore_eos, seed=sampling.resolved_seed())
         self.scheduler.add(request)

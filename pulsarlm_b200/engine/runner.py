@@ -42,7 +42,7 @@ class StepEntry:
 
 
 STATUS_MESSAGES = {
-    1: "a token id outside the vocabulary reached the embedding kernel",
+    1: "a token id outside the vocabulary, or a position past the model's table, reached the embedding kernel",
     2: "a token's block-table entry was not a page of the pool when its key was written",
     4: "a block-table entry was not a page of the pool when attention read it",
     8: "a bounded wait inside a kernel gave up (a barrier or a copy that never arrived)",
@@ -163,6 +163,12 @@ class ModelRunner:
                     raise ValueError(f"request {e.request!r}: token id {bad[0]} is outside [0, {self.vocab})")
             if e.want and not all(0 <= w < n for w in e.want):
                 raise ValueError(f"request {e.request!r}: wanted places {e.want} are outside its {n} tokens")
+        limit = self.model.spec.max_positions
+        if limit is not None:
+            for e in entries:
+                held = self.cache.length(e.request) if self.cache.is_open(e.request) else 0
+                if held + len(e.tokens) > limit:
+                    raise ValueError(f"request {e.request!r}: {held + len(e.tokens)} tokens exceed the model's {limit} positions")
         for e in entries:
             if not self.cache.is_open(e.request):
                 if self.cache.open(e.request) is None:

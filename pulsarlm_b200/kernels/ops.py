@@ -25,7 +25,7 @@ _PTR = ctypes.c_void_p
 _lib = None
 _lock = threading.Lock()
 
-ABI_VERSION = 30
+ABI_VERSION = 31
 
 DTYPE_CODE = {torch.float32: 0, torch.bfloat16: 1}
 
@@ -54,7 +54,7 @@ _SIGNATURES = {
                          _PTR, _I32, _I32, _I32, _I32, _I32, _I32, _PTR, _PTR, _F32, _PTR, _PTR],
     "pl_attention_simt": [_PTR, _I64, _PTR, _PTR, _I64, _I64, _I32, _I32, _PTR, _I32, _PTR, _PTR, _PTR, _I64,
                           _I32, _I32, _I32, _I32, _I32, _F32, _F32, _I32, _PTR, _PTR, _PTR, _PTR, _PTR, _I64, _PTR,
-                          _I32, _PTR, _PTR, _PTR],
+                          _I32, _PTR, _I32, _PTR, _PTR],
     "pl_attention_decode": [_PTR, _I64, _PTR, _PTR, _I64, _I64, _I32, _I32, _PTR, _I32, _PTR, _PTR, _PTR, _I64,
                             _I32, _I32, _I32, _I32, _I32, _F32, _I32, _PTR, _PTR, _PTR, _PTR],
     "pl_attention_decode_mass": [_PTR, _I64, _PTR, _PTR, _I64, _I64, _I32, _I32, _PTR, _I32, _PTR, _PTR, _PTR, _I64,
@@ -80,6 +80,8 @@ _SIGNATURES = {
     "pl_attention_prefill_tcgen05_slopes": [_PTR, _I64, _I32, _PTR, _PTR, _I64, _I64, _I32, _I32, _PTR, _I32, _PTR,
                                             _I32, _PTR, _I64, _I32, _I32, _I32, _I32, _F32, _I32, _PTR, _PTR, _PTR,
                                             _PTR, _PTR],
+    "pl_attention_prefill_tcgen05_reach": [_PTR, _I64, _I32, _PTR, _PTR, _I64, _I64, _I32, _I32, _PTR, _I32, _PTR, _I32,
+                                           _PTR, _I64, _I32, _I32, _I32, _I32, _F32, _I32, _PTR, _PTR, _I32, _PTR, _PTR],
     "pl_attention_prefill_tcgen05_tile_rows": [_I32],
     "pl_attention_prefill_tcgen05_supports": [_I32, _I32, _I32, _I64, _I64, _I64, _I32],
     "pl_attention_prefill_tile_rows": [],
@@ -100,11 +102,11 @@ _SIGNATURES = {
     "pl_short_conv_state_strided": [_PTR, _I64, _PTR, _PTR, _PTR, _I32, _I32, _I32, _I32, _PTR],
     "pl_gated_delta": [_PTR, _PTR, _PTR, _I64, _PTR, _I64, _PTR, _I64, _PTR, _I64, _PTR, _PTR, _PTR, _PTR, _PTR, _PTR,
                        _PTR, _PTR, _PTR, _I64, _I32, _I32, _I32, _I32, _I32, _I32, _F32, _F32, _F32, _I32, _PTR],
-    "pl_moe_route": [_PTR, _I64, _PTR, _PTR, _PTR, _PTR, _I32, _I32, _I32, _I32, _I32, _I32, _I32, _I32, _I32, _PTR,
+    "pl_moe_route": [_PTR, _I64, _PTR, _PTR, _PTR, _PTR, _PTR, _I32, _I32, _I32, _I32, _I32, _I32, _I32, _I32, _I32, _PTR,
                      _I32, _PTR],
-    "pl_moe_up": [_PTR, _I64, _PTR, _PTR, _PTR, _I32, _I32, _I32, _I32, _I32, _I32, _PTR],
-    "pl_pair_embed": [_PTR, _PTR, _PTR, _PTR, _PTR, _PTR, _PTR, _PTR, _I32, _I32, _I32, _I32, _I64, _I64, _I32, _I32,
-                      _PTR, _PTR],
+    "pl_moe_up": [_PTR, _I64, _PTR, _PTR, _PTR, _I32, _I32, _I32, _I32, _I32, _I32, _I32, _PTR],
+    "pl_pair_embed": [_PTR, _PTR, _PTR, _PTR, _PTR, _PTR, _PTR, _PTR, _I32, _I32, _I32, _I32, _I64, _I64, _I32, _F32,
+                      _PTR, _I32, _I32, _PTR, _PTR],
     "pl_pair_embed_state": [_PTR, _PTR, _PTR, _PTR, _I32, _PTR],
     "pl_norm_rope_mix_write": [_PTR, _PTR, _PTR, _I64, _PTR, _I64, _F32, _PTR, _PTR, _PTR, _PTR, _I32, _PTR, _PTR,
                                _I64, _I64, _I32, _I32, _PTR, _I32, _I32, _I32, _I32, _I32, _I32, _I32, _I32, _PTR,
@@ -134,6 +136,18 @@ _SIGNATURES = {
                        _PTR, _PTR, _I32, _I32, _I32, _I32, _I32, _I32, _PTR],
     "pl_linear_step": [_PTR, _I64, _PTR, _PTR, _PTR, _I32, _PTR, _PTR, _PTR, _PTR, _PTR, _PTR, _I64, _PTR, _PTR, _PTR,
                        _PTR, _PTR, _PTR, _I32, _I32, _I32, _PTR],
+    "pl_latent_norms": [_PTR, _I64, _PTR, _I32, _PTR, _PTR, _I64, _PTR, _I32, _F32, _PTR, _PTR, _PTR, _I32, _PTR, _I64,
+                        _I32, _I32, _I32, _I32, _PTR, _PTR],
+    "pl_matrix_memory_head_floats": [_I32, _I32],
+    "pl_matrix_memory_chunk_tokens": [],
+    "pl_matrix_memory_chunks_supports": [_I32, _I32, _I32],
+    "pl_matrix_memory_step_supports": [_I32, _I32, _I32, _I32],
+    "pl_matrix_memory_walk": [_PTR, _PTR, _PTR, _PTR, _I64, _PTR, _PTR, _PTR, _F32, _PTR, _F32, _F32, _PTR, _PTR, _PTR,
+                              _PTR, _PTR, _PTR, _PTR, _PTR, _I32, _I32, _I32, _I32, _I32, _I32, _PTR],
+    "pl_matrix_memory_chunks": [_PTR, _PTR, _PTR, _PTR, _I64, _PTR, _PTR, _PTR, _F32, _PTR, _F32, _F32, _PTR, _PTR, _PTR,
+                                _I32, _PTR, _I32, _PTR, _PTR, _PTR, _PTR, _I32, _I32, _I32, _PTR],
+    "pl_matrix_memory_step": [_PTR, _PTR, _PTR, _PTR, _I64, _PTR, _I64, _I32, _PTR, _PTR, _PTR, _F32, _PTR, _F32, _F32,
+                              _PTR, _PTR, _PTR, _PTR, _I32, _I32, _I32, _I32, _PTR],
     "pl_capped_scale": [_PTR, _I64, _F32, _F32, _PTR],
     "pl_sample": [_PTR, _I64, _I32, _I32, _PTR, _PTR, _PTR, _PTR, _PTR, _PTR, _PTR],
 }
@@ -274,12 +288,14 @@ def take_tokens(tokens: torch.Tensor, source: torch.Tensor, ids: torch.Tensor,
 
 def pair_embed(table: torch.Tensor, pairs: torch.Tensor, tokens: torch.Tensor, pos: torch.Tensor, entry: torch.Tensor,
                slots: torch.Tensor, last_token: torch.Tensor, out: torch.Tensor, mul_prev: int, mul_cur: int,
-               single_tokens: bool, status: torch.Tensor | None = None) -> None:
-    """out[t] (fp32 [T, H]) = table[tokens[t]] + pairs[(before * mul_prev + tokens[t] * mul_cur) mod buckets], with
+               single_tokens: bool, status: torch.Tensor | None = None, scale: float = 1.0,
+               places: torch.Tensor | None = None) -> None:
+    """out[t] (fp32 [T, H]) = table[tokens[t]] * scale (+ places[pos[t]] where given, [positions, H]) + pairs[(before * mul_prev + tokens[t] * mul_cur) mod buckets], with
     pairs [buckets + 1, H] and its last row for a token at position 0. The token before row t is the row above it
     where that is the same entry's, else last_token[slots[entry[t]]] (int32, one per request slot), which afterwards
     holds the entry's last token (single_tokens: every entry brings one token and one launch does both)."""
-    _dev(table, pairs, tokens, pos, entry, slots, last_token, out, status)
+    _dev(table, pairs, tokens, pos, entry, slots, last_token, out, status, places)
+    assert places is None or (places.is_contiguous() and places.dtype == table.dtype and places.shape[1] == table.shape[1])
     assert table.is_contiguous() and pairs.is_contiguous() and out.is_contiguous() and out.dtype == torch.float32
     assert table.dtype == pairs.dtype and table.shape[1] == pairs.shape[1] == out.shape[1] and pairs.shape[0] >= 2
     for t in (tokens, pos, entry, slots, last_token):
@@ -288,7 +304,8 @@ def pair_embed(table: torch.Tensor, pairs: torch.Tensor, tokens: torch.Tensor, p
     assert pos.numel() == n and entry.numel() == n and out.shape[0] == n
     vocab, hidden = table.shape
     _call("pl_pair_embed", _p(table), _p(pairs), _p(tokens), _p(pos), _p(entry), _p(slots), _p(last_token), _p(out), n,
-          hidden, vocab, pairs.shape[0] - 1, int(mul_prev), int(mul_cur), int(bool(single_tokens)), _code(table.dtype),
+          hidden, vocab, pairs.shape[0] - 1, int(mul_prev), int(mul_cur), int(bool(single_tokens)), float(scale),
+          _p(places), places.shape[0] if places is not None else 0, _code(table.dtype),
           _p(status), _stream())
     if not single_tokens:
         _call("pl_pair_embed_state", _p(tokens), _p(entry), _p(slots), _p(last_token), n, _stream())
@@ -396,11 +413,11 @@ def add_normed_rmsnorm(x: torch.Tensor, y: torch.Tensor, y_weight: torch.Tensor,
           _code(y.dtype), _stream())
 
 
-BIAS_ACT = {"none": 0, "relu2": 1, "tanh": 2}
+BIAS_ACT = {"none": 0, "relu2": 1, "tanh": 2, "gelu": 3}
 
 
 def bias_act(x: torch.Tensor, bias: torch.Tensor | None, out: torch.Tensor, act: str = "none") -> None:
-    """out = act(x + bias) over [T, N]; act "none", "relu2" (the square of relu) or "tanh". x may be
+    """out = act(x + bias) over [T, N]; act "none", "relu2" (the square of relu), "tanh" or "gelu" (the exact one). x may be
     columns of a wider matrix (row stride free); out is dense and may be x."""
     _dev(x, bias, out)
     tokens, width = x.shape
@@ -605,29 +622,32 @@ def gated_delta(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, b_pre: torch.
 
 def moe_route(h: torch.Tensor, router: torch.Tensor, correction: torch.Tensor | None, top: int, n_groups: int,
               keep: int, sigmoid_scores: bool = False, group_top: int = 1, renormalise: bool = True,
-              shared_weights: torch.Tensor | None = None) -> tuple[torch.Tensor, torch.Tensor]:
+              shared_weights: torch.Tensor | None = None, logit_bias: torch.Tensor | None = None) -> tuple[torch.Tensor, torch.Tensor]:
     """(ids int32 [T, top], weights fp32 [T, top]) of the experts each token's router chooses (see csrc/moe.cu).
     sigmoid_scores: scores are sigmoids of the logits instead of their softmax; group_top: how many of a
     group's largest choice scores add up to its score; renormalise: the chosen scores over their sum. shared_weights
-    (fp32 [T]): the router's last row is no expert's but a shared expert's gate, and its sigmoid goes there."""
-    _dev(h, router, correction, shared_weights)
+    (fp32 [T]): the router's last row is no expert's but a shared expert's gate, and its sigmoid goes there. logit_bias
+    (fp32 [E]) joins the experts' logits."""
+    _dev(h, router, correction, shared_weights, logit_bias)
     tokens, hidden = h.shape
     n_experts = router.shape[0] - (1 if shared_weights is not None else 0)
     assert router.dtype == torch.float32 and router.shape[1] == hidden and router.is_contiguous() and n_experts > 0
     assert shared_weights is None or (shared_weights.dtype == torch.float32 and shared_weights.shape == (tokens,)
                                       and shared_weights.is_contiguous())
-    assert correction is None or (correction.dtype == torch.float32 and correction.shape == (n_experts,))
+    for v in (correction, logit_bias):
+        assert v is None or (v.dtype == torch.float32 and v.shape == (n_experts,) and v.is_contiguous())
     assert h.stride(1) == 1
     ids = torch.empty((tokens, top), dtype=torch.int32, device=h.device)
     weights = torch.empty((tokens, top), dtype=torch.float32, device=h.device)
-    _call("pl_moe_route", _p(h), h.stride(0) if tokens > 1 else hidden, _p(router), _p(correction), _p(ids),
+    _call("pl_moe_route", _p(h), h.stride(0) if tokens > 1 else hidden, _p(router), _p(logit_bias), _p(correction), _p(ids),
           _p(weights), tokens, hidden, n_experts, top, n_groups, keep, int(bool(sigmoid_scores)), int(group_top),
           int(bool(renormalise)), _p(shared_weights), _code(h.dtype), _stream())
     return ids, weights
 
 
-def moe_up(h: torch.Tensor, up: torch.Tensor, ids: torch.Tensor, act: torch.Tensor) -> None:
-    """act[t * top + j] = relu(Wu h_t)^2 with the weights of expert ids[t, j]; up [E, ff, H] (experts without a gate)."""
+def moe_up(h: torch.Tensor, up: torch.Tensor, ids: torch.Tensor, act: torch.Tensor, activation: str = "relu2") -> None:
+    """act[t * top + j] = a(Wu h_t) with the weights of expert ids[t, j]; up [E, ff, H] (experts without a gate);
+    activation "relu2" or "gelu" (the exact one)."""
     _dev(h, up, ids, act)
     tokens, hidden = h.shape
     n_experts, ff, _ = up.shape
@@ -635,7 +655,7 @@ def moe_up(h: torch.Tensor, up: torch.Tensor, ids: torch.Tensor, act: torch.Tens
     assert up.is_contiguous() and up.shape[2] == hidden and up.dtype == h.dtype == act.dtype
     assert act.is_contiguous() and act.shape == (tokens * top, ff) and ids.is_contiguous() and h.stride(1) == 1
     _call("pl_moe_up", _p(h), h.stride(0) if tokens > 1 else hidden, _p(up), _p(ids), _p(act), tokens, hidden, ff, top,
-          n_experts, _code(h.dtype), _stream())
+          n_experts, BIAS_ACT[activation], _code(h.dtype), _stream())
 
 
 def moe_gate_up(h: torch.Tensor, gate_up: torch.Tensor, ids: torch.Tensor, act: torch.Tensor,
@@ -724,6 +744,28 @@ def norm_write_paged(z: torch.Tensor, weight: torch.Tensor, eps: float, pos: tor
     _call("pl_norm_write_paged", _p(z), z.stride(0), _p(weight), float(eps), _p(pos), _p(entry), _p(table),
           table.shape[1], _p(pool), pool.stride(0), page_size, pool.shape[0], rank, tokens, _code(z.dtype),
           _p(status), _stream())
+
+
+def latent_norms(query_z: torch.Tensor, query_weight: torch.Tensor, query_out: torch.Tensor, z: torch.Tensor | None,
+                 weight: torch.Tensor | None, eps: float, pos: torch.Tensor, entry: torch.Tensor, table: torch.Tensor,
+                 pool: torch.Tensor | None, page_size: int, status: torch.Tensor | None = None) -> None:
+    """query_out = rmsnorm(query_z) * query_weight (dense [T, query_rank]) and, where z is given, norm_write_paged of z
+    in the same launch; query_z and z have free row strides."""
+    _dev(query_z, query_weight, query_out, z, weight, pos, entry, table, pool, status)
+    tokens, query_rank = query_z.shape
+    assert query_z.stride(1) == 1 and query_weight.dtype == torch.float32 and query_weight.shape == (query_rank,)
+    assert query_weight.is_contiguous() and query_out.is_contiguous() and query_out.shape == query_z.shape
+    assert query_out.dtype == query_z.dtype and table.dim() == 2 and table.is_contiguous()
+    rank = 0
+    if z is not None:
+        rank = z.shape[1]
+        assert z.shape[0] == tokens and z.stride(1) == 1 and z.dtype == query_z.dtype and pool.dtype == z.dtype
+        assert weight.dtype == torch.float32 and weight.shape == (rank,) and weight.is_contiguous()
+        assert pool.shape[1:] == (1, page_size, rank) and pool.stride(3) == 1 and pool.stride(2) == rank
+    _call("pl_latent_norms", _p(query_z), query_z.stride(0), _p(query_weight), query_rank, _p(query_out), _p(z),
+          z.stride(0) if z is not None else 0, _p(weight) if z is not None else None, rank, float(eps), _p(pos), _p(entry),
+          _p(table), table.shape[1], _p(pool), pool.stride(0) if pool is not None else 0, page_size,
+          pool.shape[0] if pool is not None else 0, tokens, _code(query_z.dtype), _p(status), _stream())
 
 
 def add_layernorm(x: torch.Tensor, y: torch.Tensor | None, y_weight: torch.Tensor | None,
@@ -1005,6 +1047,115 @@ def linear_step(x: torch.Tensor, row_stride: int, x_bias: torch.Tensor, weight: 
           _p(out), tokens, width, block, _stream())
 
 
+def matrix_memory_head_floats(dim: int, vdim: int) -> int:
+    """Floats a head of the matrix memory keeps per request: the state [dim, vdim], the normaliser [dim], the
+    stabiliser, padding to a multiple of four."""
+    return (dim * vdim + dim + 1 + 3) // 4 * 4
+
+
+def matrix_memory_chunk_tokens() -> int:
+    return int(library().pl_matrix_memory_chunk_tokens())
+
+
+def matrix_memory_chunks_supports(dim: int, vdim: int, dtype: torch.dtype) -> bool:
+    """Whether the chunked kernels take portions of this shape."""
+    return bool(library().pl_matrix_memory_chunks_supports(dim, vdim, DTYPE_CODE.get(dtype, -1)))
+
+
+def matrix_memory_step_supports(dim: int, vdim: int, hidden: int, dtype: torch.dtype) -> bool:
+    """Whether the single-token kernel takes this shape."""
+    return bool(library().pl_matrix_memory_step_supports(dim, vdim, hidden, DTYPE_CODE.get(dtype, -1)))
+
+
+def _memory_columns(columns: tuple, heads: int, dim: int, vdim: int) -> None:
+    q, k, v, g = columns
+    assert q.shape == k.shape and q.shape[1] == heads * dim and v.shape == g.shape == (q.shape[0], heads * vdim)
+    for x in columns:
+        assert x.dtype == q.dtype and x.stride(1) == 1
+
+
+def _memory_constants(gate_bias: tuple, norm: torch.Tensor, states: torch.Tensor, heads: int, dim: int, vdim: int) -> None:
+    for b in gate_bias:
+        assert b.dtype == torch.float32 and b.shape == (heads,) and b.is_contiguous()
+    assert norm.dtype == torch.float32 and norm.shape == (heads * vdim,) and norm.is_contiguous()
+    assert states.dtype == torch.float32 and states.is_contiguous()
+    assert states.shape[1:] == (heads, matrix_memory_head_floats(dim, vdim))
+
+
+def matrix_memory_walk(columns: tuple, row_stride: int, logits: torch.Tensor, gate_bias: tuple, cap: float,
+                       norm: torch.Tensor, eps: float, q_scale: float, states: torch.Tensor, first: torch.Tensor,
+                       count: torch.Tensor, slots: torch.Tensor, entry: torch.Tensor, out: torch.Tensor, heads: int,
+                       dim: int, vdim: int) -> None:
+    """The matrix memory with exponential gates over each entry's rows, one token after the other (csrc/matrix_memory.cu).
+    columns: (q, k [T, heads * dim], v, g [T, heads * vdim]) of one matrix whose rows are row_stride elements apart;
+    logits fp32 [T, 2 * heads] (input gates, then forget gates); gate_bias: (input, forget) fp32 [heads]; states fp32
+    [slots, heads, matrix_memory_head_floats] is updated; out [T, heads * vdim]: normed and gated."""
+    q, k, v, g = columns
+    _dev(q, k, v, g, logits, *gate_bias, norm, states, first, count, slots, entry, out)
+    _memory_columns(columns, heads, dim, vdim)
+    _memory_constants(gate_bias, norm, states, heads, dim, vdim)
+    tokens = q.shape[0]
+    assert logits.dtype == torch.float32 and logits.shape == (tokens, 2 * heads) and logits.is_contiguous()
+    assert out.is_contiguous() and out.shape == v.shape and out.dtype == q.dtype
+    for x in (first, count, slots, entry):
+        assert x.dtype == torch.int32 and x.is_contiguous()
+    assert entry.numel() == tokens and first.numel() == count.numel() <= slots.numel()
+    raw = torch.empty((tokens, heads, vdim + 1), dtype=torch.float32, device=q.device)
+    top = torch.empty((tokens, heads), dtype=torch.float32, device=q.device)
+    _call("pl_matrix_memory_walk", _p(q), _p(k), _p(v), _p(g), row_stride, _p(logits), _p(gate_bias[0]), _p(gate_bias[1]),
+          float(cap), _p(norm), float(eps), float(q_scale), _p(states), _p(first), _p(count), _p(slots), _p(entry), _p(raw),
+          _p(top), _p(out), tokens, first.numel(), heads, dim, vdim, _code(q.dtype), _stream())
+    global _launches
+    _launches += 1  # (two kernels)
+
+
+def matrix_memory_chunks(columns: tuple, row_stride: int, logits: torch.Tensor, gate_bias: tuple, cap: float,
+                         norm: torch.Tensor, eps: float, q_scale: float, states: torch.Tensor, slots: torch.Tensor,
+                         chunks: torch.Tensor, spans: torch.Tensor, out: torch.Tensor, heads: int, dim: int,
+                         vdim: int) -> None:
+    """matrix_memory_walk for bfloat16 portions, in chunks on tensor cores. chunks int32 [n, 4]: {first row, rows, entry,
+    1 on the entry's last chunk}; spans int32 [m, 4]: {first chunk, chunks, entry, 0}, an entry each. Rows that no chunk
+    lists are left alone."""
+    q, k, v, g = columns
+    _dev(q, k, v, g, logits, *gate_bias, norm, states, slots, chunks, spans, out)
+    _memory_columns(columns, heads, dim, vdim)
+    _memory_constants(gate_bias, norm, states, heads, dim, vdim)
+    assert q.dtype == torch.bfloat16 == out.dtype
+    assert logits.dtype == torch.float32 and logits.shape == (q.shape[0], 2 * heads) and logits.is_contiguous()
+    assert out.is_contiguous() and out.shape == v.shape and slots.dtype == torch.int32 and slots.is_contiguous()
+    for x in (chunks, spans):
+        assert x.dtype == torch.int32 and x.dim() == 2 and x.shape[1] == 4 and x.is_contiguous()
+    n = chunks.shape[0]
+    sums = torch.empty((n, heads, matrix_memory_head_floats(dim, vdim)), dtype=torch.float32, device=q.device)
+    ends = torch.empty((n, heads, 3), dtype=torch.float32, device=q.device)  # (ends, then starts)
+    starts = ends.view(-1)[2 * n * heads:]
+    _call("pl_matrix_memory_chunks", _p(q), _p(k), _p(v), _p(g), row_stride, _p(logits), _p(gate_bias[0]),
+          _p(gate_bias[1]), float(cap), _p(norm), float(eps), float(q_scale), _p(states), _p(slots), _p(chunks), n,
+          _p(spans), spans.shape[0], _p(sums), _p(ends), _p(starts), _p(out), heads, dim, vdim, _stream())
+    global _launches
+    _launches += 2  # (three kernels)
+
+
+def matrix_memory_step(columns: tuple, row_stride: int, h: torch.Tensor, gates: torch.Tensor, gate_bias: tuple, cap: float,
+                       norm: torch.Tensor, eps: float, q_scale: float, states: torch.Tensor, slots: torch.Tensor,
+                       entry: torch.Tensor, out: torch.Tensor, heads: int, dim: int, vdim: int) -> None:
+    """matrix_memory_walk for bfloat16 steps (or leading rows) of one token per entry, in one launch. h [T, H] with gates
+    [2 * heads, H] (the input gates' rows, then the forget gates'): the gate logits are formed here, in fp32."""
+    q, k, v, g = columns
+    _dev(q, k, v, g, h, gates, *gate_bias, norm, states, slots, entry, out)
+    _memory_columns(columns, heads, dim, vdim)
+    _memory_constants(gate_bias, norm, states, heads, dim, vdim)
+    tokens, hidden = h.shape
+    assert q.dtype == torch.bfloat16 == out.dtype == h.dtype == gates.dtype and q.shape[0] == tokens
+    assert gates.shape == (2 * heads, hidden) and gates.is_contiguous() and h.stride(1) == 1
+    assert out.is_contiguous() and out.shape == v.shape
+    for x in (slots, entry):
+        assert x.dtype == torch.int32 and x.is_contiguous()
+    _call("pl_matrix_memory_step", _p(q), _p(k), _p(v), _p(g), row_stride, _p(h), h.stride(0) if tokens > 1 else hidden, hidden,
+          _p(gates), _p(gate_bias[0]), _p(gate_bias[1]), float(cap), _p(norm), float(eps), float(q_scale), _p(states),
+          _p(slots), _p(entry), _p(out), tokens, heads, dim, vdim, _stream())
+
+
 def capped_scale(x: torch.Tensor, scale: float, cap: float) -> None:
     """x (fp32, contiguous) = cap * tanh(x * scale / cap), in place."""
     _dev(x)
@@ -1175,7 +1326,8 @@ def attention_simt(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, 
                    scale: float, status: torch.Tensor | None = None, mass_sum: torch.Tensor | None = None,
                    weight_sum: torch.Tensor | None = None, query_weights: torch.Tensor | None = None,
                    softcap: float = 0.0, sinks: torch.Tensor | None = None, gate: torch.Tensor | None = None,
-                   distance_bias: torch.Tensor | None = None, distance_slopes: torch.Tensor | None = None) -> None:
+                   distance_bias: torch.Tensor | None = None, distance_slopes: torch.Tensor | None = None,
+                   keep_first: int = 0) -> None:
     """Causal paged attention; q and out [T, nh, hd] (row strides free), pools
     [pages, nkv, page_size, hd]. With mass_sum fp32 [pages, nh] and weight_sum fp32
     [pages], the attention mass of every attended page is added to them
@@ -1185,7 +1337,7 @@ def attention_simt(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, 
     stride free): head h's output for token t is multiplied by sigmoid(gate[t, h]). distance_bias
     fp32 [nh, rows]: entry min(distance, rows - 1) of a head's row is added to its scaled scores of a
     key `distance` tokens before the query. distance_slopes fp32 [nh]: slopes[h] * distance is taken off head h's
-    scaled scores."""
+    scaled scores. keep_first: a request's first keys that stay in reach besides the window's."""
     _dev(q, k_pool, v_pool, table, pos, entry, out, status, mass_sum, weight_sum, query_weights, sinks, gate,
          distance_bias, distance_slopes)
     if distance_slopes is not None:
@@ -1218,7 +1370,8 @@ def attention_simt(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, 
           n_heads, n_kv, head_dim, int(window or 0), float(scale), float(softcap or 0.0), _code(q.dtype),
           _p(mass_sum), _p(weight_sum), _p(query_weights), _p(sinks), _p(gate),
           gate.stride(0) if gate is not None else 0, _p(distance_bias),
-          distance_bias.shape[1] if distance_bias is not None else 0, _p(distance_slopes), _p(status), _stream())
+          distance_bias.shape[1] if distance_bias is not None else 0, _p(distance_slopes), int(keep_first), _p(status),
+          _stream())
 
 
 def attention_decode_supports(head_dim: int, group: int, page_size: int, dtype: torch.dtype) -> bool:
@@ -1307,22 +1460,23 @@ def attention_decode_ctas_per_sm(head_dim: int) -> int:
 
 class _AttentionExtras(ctypes.Structure):
     _fields_ = [("sinks", _PTR), ("gate", _PTR), ("gate_row_stride", _I64), ("split_weights", _I32),
-                ("softcap", _F32), ("distance_bias", _PTR), ("bias_rows", _I32), ("distance_slopes", _PTR)]
+                ("softcap", _F32), ("distance_bias", _PTR), ("bias_rows", _I32), ("distance_slopes", _PTR),
+                ("keep_first", _I32)]
 
 
 def attention_extras(q: torch.Tensor, sinks: torch.Tensor | None, gate: torch.Tensor | None,
                      split_weights: bool, softcap: float = 0.0, distance_bias: torch.Tensor | None = None,
-                     distance_slopes: torch.Tensor | None = None) -> "_AttentionExtras | None":
+                     distance_slopes: torch.Tensor | None = None, keep_first: int = 0) -> "_AttentionExtras | None":
     """What the tensor-core attention kernels take beyond plain softmax attention (the struct
     PlAttentionExtras): sinks fp32 [nh] (exp(sinks[h]) joins head h's denominator), gate [T, nh]
     logits in q's dtype (outputs times their sigmoid), split_weights (softmax weights enter the
     value product as two bfloat16 terms), softcap (> 0: scaled scores pass through softcap *
     tanh(s / softcap)), distance_bias fp32 [nh, rows] (entry min(distance, rows - 1) of a head's row joins
     its scaled scores of a key `distance` tokens before the query), distance_slopes fp32 [nh] (slopes[h] * distance
-    is taken off head h's scaled scores). None when nothing is asked for. The tensors must outlive the call that takes
+    is taken off head h's scaled scores), keep_first (a request's first keys that stay in reach besides a window's). None when nothing is asked for. The tensors must outlive the call that takes
     the struct."""
     if sinks is None and gate is None and not split_weights and not softcap and distance_bias is None \
-            and distance_slopes is None:
+            and distance_slopes is None and not keep_first:
         return None
     _dev(sinks, gate, distance_bias, distance_slopes)
     if distance_slopes is not None:
@@ -1337,7 +1491,7 @@ def attention_extras(q: torch.Tensor, sinks: torch.Tensor | None, gate: torch.Te
         assert gate.dtype == q.dtype and gate.shape == (q.shape[0], q.shape[1]) and gate.stride(1) == 1
     return _AttentionExtras(_p(sinks), _p(gate), gate.stride(0) if gate is not None else 0, int(bool(split_weights)),
                             float(softcap or 0.0), _p(distance_bias),
-                            distance_bias.shape[1] if distance_bias is not None else 0, _p(distance_slopes))
+                            distance_bias.shape[1] if distance_bias is not None else 0, _p(distance_slopes), int(keep_first))
 
 
 def attention_decode(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, table: torch.Tensor,
@@ -1467,11 +1621,13 @@ def attention_prefill_tcgen05(q: torch.Tensor, k_pool: torch.Tensor, v_pool: tor
                               scale: float, status: torch.Tensor | None = None, n_splits: int = 1,
                               scratch: torch.Tensor | None = None, wide: bool = False,
                               mass: tuple | None = None, distance_bias: torch.Tensor | None = None,
-                              distance_slopes: torch.Tensor | None = None, sinks: torch.Tensor | None = None) -> None:
+                              distance_slopes: torch.Tensor | None = None, sinks: torch.Tensor | None = None,
+                              keep_first: int = 0) -> None:
     """As attention_prefill, on the tcgen05 tensor cores. `distance_bias` fp32 [nh, rows] (even GQA groups, no
     wide tiles, no mass): entry min(distance, rows - 1) of a head's row joins its scaled scores. `distance_slopes` fp32
     [nh] (no mass; an odd group takes narrow and wide tiles alike): slopes[h] * distance is taken off head h's scaled
-    scores, and `sinks` fp32 [nh], with slopes only, join the denominators as exp(sinks[h]). With n_splits > 1 every tile's
+    scores. `sinks` fp32 [nh] (no mass, no table) join the denominators as exp(sinks[h]); keep_first (with a window;
+    no mass, nothing by distance): a request's first keys that stay in reach besides the window's. With n_splits > 1 every tile's
     keys are shared out over that many CTAs and merged through `scratch` (float32,
     attention_prefill_scratch_floats elements): for few tiles over many keys. `wide`: the
     tiles have up to attention_prefill_tcgen05_tile_rows(group) rows instead of 128.
@@ -1515,7 +1671,15 @@ def attention_prefill_tcgen05(q: torch.Tensor, k_pool: torch.Tensor, v_pool: tor
               out.stride(0), n_heads, n_kv, head_dim, int(window or 0), float(scale), int(n_splits), _p(scratch),
               _p(distance_slopes), _p(sinks), _p(status), _stream())
         return
-    assert sinks is None
+    if sinks is not None or keep_first:
+        _dev(sinks)
+        assert mass is None and distance_bias is None
+        assert sinks is None or (sinks.dtype == torch.float32 and sinks.shape == (n_heads,) and sinks.is_contiguous())
+        _call("pl_attention_prefill_tcgen05_reach", _p(q), q.stride(0), tokens, _p(k_pool), _p(v_pool), k_pool.stride(0),
+              k_pool.stride(1), page_size, n_pages, _p(table), table.shape[1], _p(tiles), tiles.shape[0], _p(out),
+              out.stride(0), n_heads, n_kv, head_dim, int(window or 0), float(scale), int(n_splits), _p(scratch),
+              _p(sinks), int(keep_first), _p(status), _stream())
+        return
     if distance_bias is not None:
         _dev(distance_bias)
         assert mass is None and not wide and (n_heads // n_kv) % 2 == 0

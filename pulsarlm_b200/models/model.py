@@ -205,6 +205,9 @@ class Model:
                     raise ValueError(
                         f"layer {layer} reads the cache of layer {src} as {want.n_kv_heads} kv heads of size "
                         f"{want.head_dim}, but it holds {have.n_kv_heads} of size {have.head_dim}")
+                if have.window is not None and want.window is not None and want.keep_first > have.keep_first:
+                    raise ValueError(f"layer {layer} reads the first {want.keep_first} tokens of layer {src}'s cache, which "
+                                     f"keeps {have.keep_first} only")
                 if have.window is not None and (want.window is None or want.window > have.window):
                     raise ValueError(
                         f"layer {layer} reads {'every key' if want.window is None else f'a window of {want.window}'} "

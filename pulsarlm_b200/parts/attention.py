@@ -207,7 +207,8 @@ class Attention(Part):
 
     params: hidden_size, n_heads, n_kv_heads, head_dim, position (a PartSpec of the
     "position" registry), scale (optional), window (optional: a query reads only
-    the last `window` keys), cache_from (optional: index of the layer whose cache
+    the last `window` keys), keep_first (optional, with a window: a sequence's first `keep_first`
+    keys stay in reach besides the window's), cache_from (optional: index of the layer whose cache
     this layer reads; it then has no k and v projections and writes nothing),
     softcap (optional: scaled scores pass through softcap * tanh(s / softcap) before
     the softmax; such a layer attends on the CUDA-core kernel, the only one that
@@ -231,6 +232,7 @@ class Attention(Part):
             raise ValueError(f"attention: {self.n_heads} heads are not a multiple of {self.n_kv} kv heads")
         self.scale = float(p["scale"]) if p.get("scale") is not None else 1.0 / math.sqrt(self.head_dim)
         self.window = int(p["window"]) if p.get("window") else None
+        self.keep_first = int(p.get("keep_first") or 0) if self.window else 0
         self.cache_from = p.get("cache_from")
         self.softcap = float(p["softcap"]) if p.get("softcap") else 0.0
         self.qk_norm_eps = float(p.get("qk_norm_eps") or 0.0)
@@ -285,11 +287,11 @@ class Attention(Part):
     def cache_need(self) -> KVCacheNeed | None:
         if self.cache_from is not None:
             return None
-        return KVCacheNeed(self.n_kv, self.head_dim, self.window, self.n_heads)
+        return KVCacheNeed(self.n_kv, self.head_dim, self.window, self.n_heads, keep_first=self.keep_first)
 
     def cache_read_need(self) -> KVCacheNeed:
         """How this layer reads a cache, its own or the one `cache_from` names."""
-        return KVCacheNeed(self.n_kv, self.head_dim, self.window, self.n_heads)
+        return KVCacheNeed(self.n_kv, self.head_dim, self.window, self.n_heads, keep_first=self.keep_first)
 
     def bind_cache(self, binding: KVBinding) -> None:
         self.cache = binding
@@ -335,7 +337,7 @@ class Attention(Part):
         and at batch 1, where sixteen CTAs rotate the same q (338 against 342 tokens/s)."""
         if not FOLD_ROPE or int(batch.n_decode) != tokens or self.cache_from is not None or inv_freq is None:
             return False
-        if rotary != self.head_dim or self.q_norm is not None or self.k_norm is not None or self.softcap:
+        if rotary != self.head_dim or self.q_norm is not None or self.k_norm is not None or self._wants_extras():
             return False
         if self.head_dim % 32 != 0:  # (the kernel rotates q in its fragments: pairs must not straddle one)
             return False
@@ -367,7 +369,7 @@ class Attention(Part):
         caller then leaves the layer to `forward`. `row_stride`: elements between the tokens'
         rows of q."""
         cache = self.cache
-        if cache is None or self.softcap or self.cache_from is not None or self.q_norm is not None \
+        if cache is None or self._wants_extras() or self.cache_from is not None or self.q_norm is not None \
                 or self.k_norm is not None or cache.mass_sum is not None:
             return None
         dtype = self.ctx.dtype
@@ -446,11 +448,19 @@ class Attention(Part):
         return self._kernels(self.ctx.dtype)[0]
 
     def _wants_extras(self) -> bool:
-        """A score cap, a sink term, a bias by distance (a table or slopes) or a gate per head: the
+        """A score cap, a sink term, kept first keys, a bias by distance (a table or slopes) or a gate per head: the
         tensor-core kernels take them in their build with extras (csrc/attention_decode.cu,
         attention_prefill.cu), without work lists or attention mass."""
         return (bool(self.softcap) or self.sinks is not None or self.distance_bias is not None or self.head_gate
-                or self.distance_slopes is not None)
+                or self.distance_slopes is not None or self.keep_first > 0)
+
+    def _reach(self, context: int, spare: int) -> int:
+        """Of `context` keys, how many a query may read: the window's (`spare` more for where its tiles start) and the
+        kept first keys' tiles."""
+        if not self.window:
+            return context
+        kept = -(-self.keep_first // spare) * spare if self.keep_first else 0
+        return min(context, self.window + spare + kept)
 
     def plan_key(self):
         """Layers of equal tiling share one plan: the tile lists depend on the kernels'
@@ -459,7 +469,8 @@ class Attention(Part):
             return None
         wide = (self.n_heads // self.n_kv) % 2 == 1
         return ("attention", self.cache.page_size, self.head_dim, self.n_heads // self.n_kv, wide,
-                self.ctx.dtype, self._wants_extras(), self.distance_slopes is not None, self.n_kv, self.window)
+                self.ctx.dtype, self._wants_extras(), self.distance_slopes is not None, self.n_kv, self.window,
+                self._reach_alone(None))
 
     def native_key(self):
         """What `native_choice` depends on beyond `plan_key`: layers that agree in both get
@@ -535,7 +546,7 @@ class Attention(Part):
             start = step.context_lens[e] - n
             for r in range(0, n, rows):
                 tiles.append((at + r, min(rows, n - r), start + r, e))
-            if wide_rows > rows and (not extras or self.distance_slopes is not None):
+            if wide_rows > rows and (not extras or self.distance_slopes is not None or self._reach_alone(None)):
                 for r in range(0, n, wide_rows):
                     wide_tiles.append((at + r, min(wide_rows, n - r), start + r, e))
         tiles.sort(key=lambda t: -(t[2] + t[1]))
@@ -558,9 +569,16 @@ class Attention(Part):
         return (self.distance_slopes is not None and gate is None and self.distance_bias is None and not self.softcap
                 and not self.split_weights)
 
+    def _reach_alone(self, gate) -> bool:
+        """Whether the layer's extras are a sink and / or kept first keys, with the softmax weights in one bfloat16 term:
+        what the tcgen05 prompt kernel's builds for those take."""
+        return ((self.sinks is not None or self.keep_first > 0) and self.distance_slopes is None
+                and self.distance_bias is None and gate is None and not self.head_gate and not self.softcap
+                and not self.split_weights)
+
     def _attend_with_extras(self, q, out, table, batch, plan, decode_kernel: bool, prefill_kernel: bool,
                             gate: torch.Tensor | None = None) -> None:
-        """Attention with a score cap, a sink term, a bias by distance and / or a gate per head
+        """Attention with a score cap, a sink term, kept first keys, a bias by distance and / or a gate per head
         (`gate`: [T, n_heads] logits). bfloat16 shapes the tensor-core
         kernels take: the leading single tokens on the split-key kernel, prompt portions on
         the tiled mma.sync kernel, both in their build with extras (cap and bias on every score
@@ -571,9 +589,7 @@ class Attention(Part):
         bias = self.distance_bias
         n_decode = min(int(batch.n_decode), tokens) if decode_kernel else 0
         if n_decode > 0:
-            max_context = plan.get("max_context") or max(batch.host_context_lens[:n_decode])
-            if self.window:
-                max_context = min(max_context, self.window + 16)
+            max_context = self._reach(plan.get("max_context") or max(batch.host_context_lens[:n_decode]), 16)
             splits = decode_splits(n_decode * self.n_kv, max_context, q.device, self.head_dim,
                                    self.n_heads // self.n_kv)
             scratch = None
@@ -587,25 +603,23 @@ class Attention(Part):
                                  extras=ops.attention_extras(q[:n_decode], self.sinks,
                                                              gate[:n_decode] if gate is not None else None,
                                                              self.split_weights, self.softcap, bias,
-                                                             self.distance_slopes))
+                                                             self.distance_slopes, self.keep_first))
         if n_decode == tokens:
             return
         tiles = plan.get("tiles")
         if prefill_kernel and tiles is not None and n_decode == int(batch.n_decode):
             # (the tile list covers exactly the tokens after the leading single tokens)
-            if self._bias_alone(gate) or self._slopes_alone(gate):
-                # A bias by distance and nothing else (or slopes, and perhaps a sink): the tcgen05 kernel's builds that
-                # add it to their products.
+            if self._bias_alone(gate) or self._slopes_alone(gate) or self._reach_alone(gate):
+                # A bias by distance and nothing else (or slopes, and perhaps a sink; or a sink and kept first keys): the
+                # tcgen05 kernel's builds for it.
                 if self._prefill_tcgen05 is None:
                     self._prefill_tcgen05 = ops.attention_prefill_tcgen05_supports(q, cache.k_pool, cache.page_size)
                 if self._prefill_tcgen05:
-                    odd = (self.n_heads // self.n_kv) % 2 == 1   # (slopes only) a head per CTA, tiles of up to twice the rows
+                    odd = (self.n_heads // self.n_kv) % 2 == 1   # (no table) a head per CTA, tiles of up to twice the rows
                     if odd and plan.get("tiles_wide") is not None:
                         tiles = plan["tiles_wide"]
                     ctas = tiles.shape[0] * (self.n_heads if odd else self.n_heads // 2)
-                    max_keys = int(plan.get("max_keys") or 0)
-                    if self.window:
-                        max_keys = min(max_keys, self.window + ops.attention_prefill_tile_rows())
+                    max_keys = self._reach(int(plan.get("max_keys") or 0), ops.attention_prefill_tile_rows())
                     splits = prefill_splits(ctas, max_keys, tokens - n_decode, self.n_heads, self.head_dim, q.device)
                     scratch = None
                     if splits > 1:
@@ -615,18 +629,18 @@ class Attention(Part):
                     ops.attention_prefill_tcgen05(q, cache.k_pool, cache.v_pool, table, tiles, out, cache.page_size,
                                                   self.window, self.scale, batch.status, splits, scratch, False,
                                                   distance_bias=bias, distance_slopes=self.distance_slopes,
-                                                  sinks=self.sinks)
+                                                  sinks=self.sinks, keep_first=self.keep_first)
                     return
             ops.attention_prefill(q, cache.k_pool, cache.v_pool, table, tiles, out, cache.page_size, self.window,
                                   self.scale, batch.status,
                                   extras=ops.attention_extras(q, self.sinks, gate, self.split_weights, self.softcap,
-                                                              bias, self.distance_slopes))
+                                                              bias, self.distance_slopes, self.keep_first))
             return
         ops.attention_simt(q[n_decode:], cache.k_pool, cache.v_pool, table, batch.pos[n_decode:],
                            batch.entry[n_decode:], out[n_decode:], cache.page_size, self.window, self.scale,
                            batch.status, softcap=self.softcap, sinks=self.sinks,
                            gate=gate[n_decode:] if gate is not None else None, distance_bias=bias,
-                           distance_slopes=self.distance_slopes)
+                           distance_slopes=self.distance_slopes, keep_first=self.keep_first)
 
     def attend(self, q: torch.Tensor, out: torch.Tensor, table: torch.Tensor, batch, rope: tuple | None = None,
                gate: torch.Tensor | None = None) -> None:
@@ -676,7 +690,7 @@ class Attention(Part):
                                    batch.status, cache.mass_sum, cache.weight_sum, weights[:n_simt],
                                    softcap=self.softcap, sinks=self.sinks,
                                    gate=gate[:n_simt] if gate is not None else None, distance_bias=self.distance_bias,
-                                   distance_slopes=self.distance_slopes)
+                                   distance_slopes=self.distance_slopes, keep_first=self.keep_first)
             if fast:
                 ops.attention_prefill_tcgen05(q, cache.k_pool, cache.v_pool, table, tiles, out, cache.page_size,
                                               self.window, self.scale, batch.status, 1, None, wide,

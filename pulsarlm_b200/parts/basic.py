@@ -354,12 +354,13 @@ class Embedding(Part):
 
 @register_part("embedding", "pair_hash_table")
 class PairHashEmbedding(Part):
-    """x[t] = weight[token[t]] + pairs[(before * mul_prev + token[t] * mul_cur) mod buckets] in fp32,
-    where `before` is the token ahead of token[t] in its sequence; a sequence's first token
+    """x[t] = weight[token[t]] * scale + pairs[(before * mul_prev + token[t] * mul_cur) mod buckets] (+ places[p],
+    a learned vector of the token's position p) in fp32, where `before` is the token ahead of token[t] in its sequence; a sequence's first token
     takes the last row of `pairs` (row number `buckets`). The token before a step's first token
     is part of the request's state: one int32 per request slot, which the kernel reads for an
     entry's first row and moves on to the entry's last token. params: vocab_size, hidden_size,
-    buckets, mul_prev, mul_cur. tensors: weight [vocab, hidden], pairs [buckets + 1, hidden]."""
+    buckets, mul_prev, mul_cur, scale (optional, 1 when absent), positions (optional: rows of `places`).
+    tensors: weight [vocab, hidden], pairs [buckets + 1, hidden], places [positions, hidden]."""
 
     def __init__(self, spec: PartSpec, ctx: BuildContext):
         super().__init__(spec, ctx)
@@ -368,6 +369,9 @@ class PairHashEmbedding(Part):
         self.buckets = int(self.param("buckets"))
         self.mul_prev = int(self.param("mul_prev"))
         self.mul_cur = int(self.param("mul_cur"))
+        self.scale = float(spec.params["scale"]) if spec.params.get("scale") is not None else 1.0
+        self.positions = int(spec.params.get("positions") or 0)
+        self.places: torch.Tensor | None = None
         if self.buckets <= 0:
             raise ValueError(f"pair_hash_table: buckets must be positive, got {self.buckets}")
         self.weight: torch.Tensor | None = None
@@ -377,12 +381,16 @@ class PairHashEmbedding(Part):
     @classmethod
     def tensor_needs(cls, spec: PartSpec) -> dict[str, TensorNeed]:
         p = spec.params
-        return {spec.tensors["weight"]: TensorNeed((int(p["vocab_size"]), int(p["hidden_size"]))),
-                spec.tensors["pairs"]: TensorNeed((int(p["buckets"]) + 1, int(p["hidden_size"])))}
+        needs = {spec.tensors["weight"]: TensorNeed((int(p["vocab_size"]), int(p["hidden_size"]))),
+                 spec.tensors["pairs"]: TensorNeed((int(p["buckets"]) + 1, int(p["hidden_size"])))}
+        if p.get("positions"):
+            needs[spec.tensors["places"]] = TensorNeed((int(p["positions"]), int(p["hidden_size"])))
+        return needs
 
     def load(self, tensors: dict[str, torch.Tensor]) -> None:
         self.weight = tensors[self.spec.tensors["weight"]].contiguous()
         self.pairs = tensors[self.spec.tensors["pairs"]].contiguous()
+        self.places = tensors[self.spec.tensors["places"]].contiguous() if self.positions else None
 
     def cache_need(self) -> StateNeed:
         return StateNeed((1,), "int32")
@@ -398,7 +406,7 @@ class PairHashEmbedding(Part):
             raise ValueError("pair_hash_table: the embedding needs the step (positions, entries, state slots)")
         x = torch.empty((tokens.numel(), self.hidden), dtype=torch.float32, device=tokens.device)
         ops.pair_embed(self.weight, self.pairs, tokens, batch.pos, batch.entry, batch.slots, self.binding.states.view(-1),
-                       x, self.mul_prev, self.mul_cur, int(batch.n_decode) == tokens.numel(), batch.status)
+                       x, self.mul_prev, self.mul_cur, int(batch.n_decode) == tokens.numel(), batch.status, self.scale, self.places)
         return x
 
 

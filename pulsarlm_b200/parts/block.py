@@ -14,7 +14,7 @@ from ..kernels import ops
 from .basic import NormedDelta, RMSNorm, ScaledPair, settle_pending
 from .branches import run_branches
 from .registry import BuildContext, build_part, register_part
-from .spec import LayerSpec
+from .spec import LayerSpec, PartSpec, TensorNeed
 
 
 @register_part("block", "pre_norm")
@@ -73,7 +73,8 @@ class SandwichNormBlock:
     Norm names in the LayerSpec: "mixer", "mixer_out", "feed_forward", "feed_forward_out".
     `extras` of the LayerSpec: "residual_mult" (m, 1 when absent) and optional PartSpecs
     "mixer_filter" / "feed_forward_filter" of the "filter" registry (e.g. a short
-    convolution over time), applied to the sublayer's input. A LayerSpec whose
+    convolution over time), applied to the sublayer's input; "ignored": {name: shape} of tensors that a checkpoint
+    may hold for the layer and nothing reads. A LayerSpec whose
     feed_forward is None has the first line only. The out-norm of a sublayer is not run
     on its own: its output travels as a NormedDelta and the next norm kernel norms it,
     adds it and norms the sum for the next sublayer in one pass."""
@@ -105,6 +106,8 @@ class SandwichNormBlock:
                     ("feed_forward", spec.feed_forward)]
             if extras.get("feed_forward_filter"):
                 out.append(("filter", extras["feed_forward_filter"]))
+        if extras.get("ignored"):
+            out.append(("block", PartSpec("ignored_tensors", {}, dict(extras["ignored"]))))
         return out
 
     def parts(self):
@@ -287,7 +290,6 @@ class ParallelBlock:
 
 
 def _scales_spec(names: dict, hidden: int):
-    from .spec import PartSpec
     return PartSpec("layer_scales", {"hidden_size": hidden}, dict(names))
 
 
@@ -309,7 +311,6 @@ class _LayerScales:
 
     @classmethod
     def tensor_needs(cls, spec):
-        from .spec import TensorNeed
         hidden = int(spec.params["hidden_size"])
         return {name: TensorNeed((hidden,), role="vector") for name in spec.tensors.values() if name}
 
@@ -317,3 +318,17 @@ class _LayerScales:
         for role, name in self.names.items():
             if name:
                 setattr(self, role, tensors[name].float().contiguous())
+
+
+@register_part("block", "ignored_tensors")
+class _IgnoredTensors:
+    """Tensors a layer's checkpoint may hold and nothing reads, as a part spec of its own so that the loader hears of
+    them. The spec's `tensors` map names to shapes."""
+
+    @classmethod
+    def part_specs(cls, spec):
+        return []
+
+    @classmethod
+    def tensor_needs(cls, spec):
+        return {name: TensorNeed(tuple(shape), role="ignored", optional=True) for name, shape in spec.tensors.items()}

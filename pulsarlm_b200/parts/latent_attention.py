@@ -52,14 +52,19 @@ class LatentAttention(Part):
     PartSpec's (`rope`: halves paired; `rope_pairs`: neighbours; its `amplitude` multiplies
     cos and sin). Without rope_dim there is no position encoding.
 
+    With `query_rank` the queries come through a latent of their own: q = Wq rmsnorm(Wdq h) * nq, Wdq the `query_down`
+    tensor [query_rank, H], nq `query_norm` [query_rank], q then [nh*(hd+r), query_rank].
+
     params: hidden_size, n_heads, head_dim (of q and k, without the rotated part), value_dim,
     latent_rank, scale, window (None: every earlier token; n: the token itself and the n - 1
     before it), eps (of the latent's norm), sink (whether the softmax has the sink term), gate
     (False; True or "head": one logit per head; "element": one per output channel), rope_dim
     and position (optional), cache_from (optional: index of the layer whose cached rows this
-    layer reads; it then has no down projection and no latent norm, and writes nothing).
+    layer reads; it then has no down projection and no latent norm, and writes nothing), query_rank
+    (optional), split_weights (optional, default true: softmax weights enter the value product in two
+    bfloat16 terms; false: in one).
     tensors: q [nh*(hd+r), H], down [rank+r, H], latent_norm [rank], up_k [nh*hd, rank],
-    up_v [nh*vd, rank], sink [nh], gate [nh, H] or [nh*vd, H], o [H, nh*vd]."""
+    up_v [nh*vd, rank], sink [nh], gate [nh, H] or [nh*vd, H], o [H, nh*vd]; query_down, query_norm."""
 
     def __init__(self, spec: PartSpec, ctx: BuildContext):
         super().__init__(spec, ctx)
@@ -79,6 +84,8 @@ class LatentAttention(Part):
         self.has_gate = self.gate_kind is not None
         self.rope_dim = int(p.get("rope_dim") or 0)
         self.row = self.rank + self.rope_dim          # what a token caches
+        self.query_rank = int(p.get("query_rank") or 0)
+        self.split_weights = bool(p.get("split_weights", True))
         self.cache_from = p.get("cache_from")
         self.position = build_part("position", p["position"], ctx) if self.rope_dim else None
         self.interleaved = bool(self.rope_dim) and p["position"].kind == "rope_pairs"
@@ -92,8 +99,12 @@ class LatentAttention(Part):
         p, t = spec.params, spec.tensors
         h, nh, hd, vd, rank = (int(p[k]) for k in ("hidden_size", "n_heads", "head_dim", "value_dim", "latent_rank"))
         rot = int(p.get("rope_dim") or 0)
-        needs = {t["q"]: TensorNeed((nh * (hd + rot), h)), t["up_k"]: TensorNeed((nh * hd, rank)),
+        query_rank = int(p.get("query_rank") or 0)
+        needs = {t["q"]: TensorNeed((nh * (hd + rot), query_rank or h)), t["up_k"]: TensorNeed((nh * hd, rank)),
                  t["up_v"]: TensorNeed((nh * vd, rank)), t["o"]: TensorNeed((h, nh * vd))}
+        if query_rank:
+            needs[t["query_down"]] = TensorNeed((query_rank, h))
+            needs[t["query_norm"]] = TensorNeed((query_rank,), role="vector")
         if p.get("cache_from") is None:
             needs[t["down"]] = TensorNeed((rank + rot, h))
             needs[t["latent_norm"]] = TensorNeed((rank,), role="vector")
@@ -106,9 +117,13 @@ class LatentAttention(Part):
     def load(self, tensors: dict[str, torch.Tensor]) -> None:
         t = self.spec.tensors
         nh, hd, vd, rank = self.n_heads, self.head_dim, self.value_dim, self.rank
-        parts = [tensors[t["q"]]] + ([tensors[t["down"]]] if self.cache_from is None else []) + (
+        first = tensors[t["query_down" if self.query_rank else "q"]]
+        parts = [first] + ([tensors[t["down"]]] if self.cache_from is None else []) + (
             [tensors[t["gate"]]] if self.has_gate else [])
-        self.stacked = torch.cat(parts, dim=0).contiguous()      # q, latent, gate logits from one product
+        self.stacked = torch.cat(parts, dim=0).contiguous()      # q (or its latent), latent, gate logits from one product
+        if self.query_rank:
+            self.query_up = tensors[t["q"]].contiguous()
+            self.query_norm = tensors[t["query_norm"]].float().contiguous()
         # q'_h = Wuk_h^T q_h as a product with rows [rank] over dim: the transposed blocks.
         self.up_k = tensors[t["up_k"]].view(nh, hd, rank).transpose(1, 2).contiguous()   # [nh, rank, hd]
         self.up_v = tensors[t["up_v"]].view(nh, vd, rank).contiguous()                   # [nh, vd, rank]
@@ -134,8 +149,20 @@ class LatentAttention(Part):
         cache = self.cache
         table = batch.tables[cache.group]
         proj = linear(h, self.stacked)
-        q = proj[:, : nh * (hd + rot)].view(tokens, nh, hd + rot)
-        at = nh * (hd + rot)
+        stored = False
+        if self.query_rank:
+            # the queries' latent, normed into a dense operand of its own product
+            at = self.query_rank
+            c_q = torch.empty((tokens, at), dtype=h.dtype, device=h.device)
+            # (without a rotated part the cached latent is normed and stored by the same launch)
+            z = proj[:, at: at + row] if self.cache_from is None and not rot else None
+            ops.latent_norms(proj[:, :at], self.query_norm, c_q, z, self.latent_norm, self.eps, batch.pos, batch.entry, table,
+                             cache.k_pool if z is not None else None, cache.page_size, batch.status)
+            stored = z is not None
+            q = linear(c_q, self.query_up).view(tokens, nh, hd + rot)
+        else:
+            q = proj[:, : nh * (hd + rot)].view(tokens, nh, hd + rot)
+            at = nh * (hd + rot)
         z = None
         if self.cache_from is None:
             z = proj[:, at: at + row]
@@ -148,7 +175,7 @@ class LatentAttention(Part):
             ops.latent_rope_write(q, q_latent, z, self.latent_norm, self.eps, rank, rot, inv_freq, self.interleaved,
                                   float(getattr(self.position, "amplitude", 1.0)), batch.pos, batch.entry, table,
                                   cache.k_pool, cache.page_size, batch.status)
-        elif z is not None:
+        elif z is not None and not stored:
             ops.norm_write_paged(z, self.latent_norm, self.eps, batch.pos, batch.entry, table, cache.k_pool,
                                  cache.page_size, batch.status)
         mixed = torch.empty((tokens, nh, row), dtype=h.dtype, device=h.device)
@@ -224,7 +251,8 @@ class LatentAttention(Part):
             if splits > 1:
                 scratch = torch.empty(ops.attention_decode_scratch_floats(n_decode, self.n_heads, self.row, splits),
                                       dtype=torch.float32, device=q.device)
-            extras = ops.attention_extras(q[:n_decode], self.sink, gate[:n_decode] if gate is not None else None, True)
+            extras = ops.attention_extras(q[:n_decode], self.sink, gate[:n_decode] if gate is not None else None,
+                                          self.split_weights)
             ops.attention_decode(q[:n_decode], cache.k_pool, cache.v_pool, table, batch.pos[:n_decode],
                                  batch.entry[:n_decode], out[:n_decode], cache.page_size, self.window, self.scale,
                                  splits, scratch, batch.status, extras=extras)
@@ -234,7 +262,7 @@ class LatentAttention(Part):
         if prefill_kernel and tiles is not None and n_decode == int(batch.n_decode):
             # (the tile list covers exactly the tokens after the leading single tokens)
             ops.attention_prefill(q, cache.k_pool, cache.v_pool, table, tiles, out, cache.page_size, self.window,
-                                  self.scale, batch.status, extras=ops.attention_extras(q, self.sink, gate, True))
+                                  self.scale, batch.status, extras=ops.attention_extras(q, self.sink, gate, self.split_weights))
             return
         ops.attention_simt(q[n_decode:], cache.k_pool, cache.v_pool, table, batch.pos[n_decode:],
                            batch.entry[n_decode:], out[n_decode:], cache.page_size, self.window, self.scale,

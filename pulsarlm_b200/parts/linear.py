@@ -157,11 +157,12 @@ ACT_IN = os.environ.get("PULSARLM_B200_ACT_IN", "1") != "0"  # (0: always the bi
 
 def activated_linear(z: torch.Tensor, bias: torch.Tensor | None, act: str, weight: torch.Tensor) -> torch.Tensor:
     """act(z + bias) W^T -> [T, N] for z [T, K] (a projection's output; its rows may be columns of a
-    wider matrix), act "relu2" or "tanh". For a handful of tokens in bfloat16 the skinny kernel forms
+    wider matrix), act "relu2", "tanh" or "gelu" (the exact one, always a kernel of its own: the skinny kernel
+    would form it anew in every tile). Else, for a handful of tokens in bfloat16 the skinny kernel forms
     the activation itself as it reads z (one launch fewer, the activation never written; the same
     bits); else the bias-and-activation kernel followed by `linear`."""
     tokens, k = z.shape
-    if (ACT_IN and z.dtype == torch.bfloat16 == weight.dtype and tokens <= ops.GEMM_GATED_IN_MAX_TOKENS
+    if (ACT_IN and act in ("relu2", "tanh") and z.dtype == torch.bfloat16 == weight.dtype and tokens <= ops.GEMM_GATED_IN_MAX_TOKENS
             and z.stride(1) == 1 and weight.stride(1) == 1 and z.data_ptr() % 16 == 0
             and own_kernel_for(tokens, weight.shape[0], z.device, k) == "skinny"
             and ops.gemm_bf16_supports(tokens, weight.shape[0], k, z.stride(0) if tokens > 1 else k, weight.stride(0))):

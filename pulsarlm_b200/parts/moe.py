@@ -1,4 +1,4 @@
-"""A routed feed-forward: many small feed-forwards (gated, or plain with the square of relu)
+"""A routed feed-forward: many small feed-forwards (gated, or plain with the square of relu or GELU)
 of which each token uses a few, chosen by a router, beside an optional one that every token uses."""
 
 from __future__ import annotations
@@ -39,7 +39,9 @@ class RoutedExperts(Part):
     (default "softmax"); `group_top` = n makes a group's score the sum of its n largest choice
     scores (default 1); `renormalise` = False leaves the chosen scores as the weights (default
     True); `expert` = "relu2" makes every expert, and the shared one, W_down relu(W_up h)^2 without
-    a gate (default "gated_silu"; such experts have no `expert_gate` / `shared_gate` tensors).
+    a gate (default "gated_silu"; such experts have no `expert_gate` / `shared_gate` tensors), "gelu" the same with the
+    exact GELU. The tensor `logit_bias` [E], where given, joins the router's logits (choice and weights see it; with
+    softmax scores and `renormalise` the weights are the softmax over the chosen experts' logits alone).
 
     `expert` = "clamped" gives experts the clamped unit in the place of silu(gate) * up (ops.gated_act) with
     `expert_limit`, and the shared expert `shared_limit`; `weigh_input` = True puts an expert's weight on its input
@@ -49,7 +51,7 @@ class RoutedExperts(Part):
 
     params: hidden_size, expert_size, n_experts, top, groups (default 1), keep_groups
     (default groups), shared_size (optional), scores, group_top, renormalise, expert, expert_limit, shared_limit,
-    weigh_input. tensors: router [E, H], correction [E]
+    weigh_input. tensors: router [E, H], correction [E] and logit_bias [E]
     (optional), experts: a name pattern with `{e}` for gate / up / down
     (`expert_gate`, `expert_up` [F, H], `expert_down` [H, F]), shared_gate, shared_up [Fs, H],
     shared_down [H, Fs]."""
@@ -68,7 +70,8 @@ class RoutedExperts(Part):
         self.group_top = int(p.get("group_top") or 1)
         self.renormalise = bool(p.get("renormalise", True))
         expert = str(p.get("expert") or "gated_silu")
-        self.gated = {"gated_silu": True, "relu2": False, "clamped": True}[expert]
+        self.gated = {"gated_silu": True, "relu2": False, "gelu": False, "clamped": True}[expert]
+        self.plain_act = "gelu" if expert == "gelu" else "relu2"   # (experts without a gate)
         self.limit = float(self.param("expert_limit")) if expert == "clamped" else None
         self.shared_limit = float(self.param("shared_limit")) if expert == "clamped" and self.shared_size else None
         self.weigh_input = bool(p.get("weigh_input", False))
@@ -80,7 +83,7 @@ class RoutedExperts(Part):
         if not 0 < self.top <= self.keep * (self.n_experts // self.groups):
             raise ValueError(f"moe: {self.top} experts cannot be chosen from {self.keep} groups of "
                              f"{self.n_experts // self.groups}")
-        self.router = self.correction = None
+        self.router = self.correction = self.logit_bias = None
         self.gate_up = self.down = None            # [E, 2F, H] ([E, F, H] without a gate), [E, H, F]
         self.gate_up_t = self.down_t = None        # the same with rows and columns swapped, for the grouped products
         self.shared_gate_up = self.shared_down = None
@@ -91,6 +94,8 @@ class RoutedExperts(Part):
         h, f, e = int(p["hidden_size"]), int(p["expert_size"]), int(p["n_experts"])
         gated = str(p.get("expert") or "gated_silu") in ("gated_silu", "clamped")
         needs = {t["router"]: TensorNeed((e, h))}
+        if t.get("logit_bias"):
+            needs[t["logit_bias"]] = TensorNeed((e,), role="offset")
         if t.get("correction"):
             needs[t["correction"]] = TensorNeed((e,), role="offset")
         for i in range(e):
@@ -114,6 +119,7 @@ class RoutedExperts(Part):
         if self.shared_gate_row:
             self.router = torch.cat([self.router, tensors[t["shared_gate_row"]].float()], dim=0).contiguous()
         self.correction = tensors[t["correction"]].float().contiguous() if t.get("correction") else None
+        self.logit_bias = tensors[t["logit_bias"]].float().contiguous() if t.get("logit_bias") else None
         experts = range(self.n_experts)
         if self.gated:
             self.gate_up = torch.stack([torch.cat([tensors[t["expert_gate"].format(e=i)],
@@ -135,7 +141,7 @@ class RoutedExperts(Part):
         """(ids, weights on the experts' inputs, weights on their outputs, weight of the shared expert); weights None: 1."""
         shared = torch.empty(h.shape[0], dtype=torch.float32, device=h.device) if self.shared_gate_row else None
         ids, weights = ops.moe_route(h, self.router, self.correction, self.top, self.groups, self.keep,
-                                     self.sigmoid_scores, self.group_top, self.renormalise, shared)
+                                     self.sigmoid_scores, self.group_top, self.renormalise, shared, self.logit_bias)
         return (ids, weights, None, shared) if self.weigh_input else (ids, None, weights, shared)
 
     def _shared(self, h: torch.Tensor) -> torch.Tensor | None:
@@ -145,7 +151,7 @@ class RoutedExperts(Part):
         if self.gated:
             act = "silu" if self.shared_limit is None else "clamped"
             return gated_feed_forward(h, self.shared_gate_up, self.shared_down, act, self.shared_limit or 0.0)
-        return activated_linear(linear(h, self.shared_gate_up), None, "relu2", self.shared_down)
+        return activated_linear(linear(h, self.shared_gate_up), None, self.plain_act, self.shared_down)
 
     def _units(self, h: torch.Tensor) -> tuple:
         """Router and first half of the chosen experts, pair by pair: (activations [T * top, F], what `_route` says)."""
@@ -154,7 +160,7 @@ class RoutedExperts(Part):
         if self.gated:
             ops.moe_gate_up(h, self.gate_up, routed[0], act, self.limit, routed[1])
         else:
-            ops.moe_up(h, self.gate_up, routed[0], act)
+            ops.moe_up(h, self.gate_up, routed[0], act, self.plain_act)
         return act, routed
 
     def forward(self, h: torch.Tensor, batch) -> torch.Tensor:
@@ -177,7 +183,7 @@ class RoutedExperts(Part):
         elif self.gated:
             ops.swiglu(gate_up, act)
         else:
-            ops.bias_act(gate_up, None, act, "relu2")
+            ops.bias_act(gate_up, None, act, self.plain_act)
         y = torch.nn.functional.grouped_mm(act, self.down.transpose(1, 2), offs=ends)
         ops.moe_combine(y, row_of_pair, weights, shared, out, shared_weights)
         return out

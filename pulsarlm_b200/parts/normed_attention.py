@@ -54,7 +54,9 @@ def bias_by_distance(table: torch.Tensor, far: float) -> torch.Tensor:
 class NormedAttention(Attention):
     """q = Wq h [heads, dim], k = Wk h [kv_heads, dim], v = Wv h [kv_heads, vdim]; causal softmax
     attention of head h over kv head h // (heads / kv_heads) with scores (q . k) * scale, an
-    optional sliding `window`, then the o projection over the concatenated heads [heads * vdim].
+    optional sliding `window` (with `keep_first`: a sequence's first keys stay in reach besides), one more term
+    exp(sink_h) in the denominator where the `sink` tensor [heads] is given, then the o projection over the
+    concatenated heads [heads * vdim].
 
     `qk_norm`: how q and k are normed (RMS, eps `norm_eps`): "per_head" over each head's dim with
     the weights `q_norm` / `k_norm` [dim] shared by the heads; "whole" over the whole projection
@@ -77,9 +79,9 @@ class NormedAttention(Attention):
     keeps the plain attention kernels in bfloat16 (tcgen05 for prompt portions at rows of 64 and
     128, work lists for many single tokens) and multiplies by the gate in a small kernel afterwards.
 
-    params: hidden_size, n_heads, n_kv_heads, head_dim (dim), value_dim, scale, window, norm_eps,
+    params: hidden_size, n_heads, n_kv_heads, head_dim (dim), value_dim, scale, window, keep_first, norm_eps,
     qk_norm, position, bias_far, bias_rows (optional), value_mix, value_stream, head_gate. tensors: q, k, v, o,
-    q_norm, k_norm, distance_bias, value_mix, gate, and `ignored`: {name: shape} of tensors that a checkpoint may
+    q_norm, k_norm, sink, distance_bias, value_mix, gate, and `ignored`: {name: shape} of tensors that a checkpoint may
     hold for the layer and nothing reads."""
 
     def __init__(self, spec: PartSpec, ctx: BuildContext):
@@ -92,7 +94,7 @@ class NormedAttention(Attention):
         super().__init__(inner, ctx)
         self.spec = spec
         if p.get("cache_from") is not None or p.get("softcap") or p.get("sink_logit") is not None:
-            raise ValueError("normed_attention: cache_from, softcap and sinks are not supported")
+            raise ValueError("normed_attention: cache_from, softcap and constant sinks are not supported")
         self.qk_norm = str(p.get("qk_norm") or "none")
         if self.qk_norm not in QK_NORMS:
             raise ValueError(f"normed_attention: unknown qk_norm {self.qk_norm!r} (known: {', '.join(QK_NORMS)})")
@@ -122,6 +124,8 @@ class NormedAttention(Attention):
         if p.get("bias_far") is not None:
             # (the table's rows are a size of the stored tensor; a configuration may name them, for random weights)
             needs[t["distance_bias"]] = TensorNeed((int(p.get("bias_rows") or -1), nh), role="offset")
+        if t.get("sink"):
+            needs[t["sink"]] = TensorNeed((nh,), role="offset")
         if p.get("head_gate"):
             needs[t["gate"]] = TensorNeed((nh, h))
         if p.get("value_mix") == "mix":
@@ -157,11 +161,13 @@ class NormedAttention(Attention):
             self.k_weight = tensors[t["k_norm"]].float().contiguous()
         if self.bias_far is not None:
             self.distance_bias = bias_by_distance(tensors[t["distance_bias"]], self.bias_far)
+        if t.get("sink"):
+            self.sinks = tensors[t["sink"]].float().contiguous()
         if self.value_mix == "mix":
             self.lam = float(tensors[t["value_mix"]].float().item())
 
     def cache_need(self) -> KVCacheNeed:
-        return KVCacheNeed(self.n_kv, self.row, self.window, self.n_heads)
+        return KVCacheNeed(self.n_kv, self.row, self.window, self.n_heads, keep_first=self.keep_first)
 
     def cache_read_need(self) -> KVCacheNeed:
         return self.cache_need()
@@ -170,7 +176,8 @@ class NormedAttention(Attention):
         super().bind_cache(binding)
         # With the cache's page size known: a gate that would be the layer's only extra stays out of the attention
         # kernels where the plain tensor-core kernels take the shape (they are the faster builds).
-        if self.gated and self.distance_bias is None and self.bias_far is None and self.ctx.dtype == torch.bfloat16:
+        if self.gated and self.distance_bias is None and self.bias_far is None and self.ctx.dtype == torch.bfloat16 \
+                and not self.spec.tensors.get("sink") and not self.keep_first:
             self._decode_kernel = self._prefill_kernel = None
             self.head_gate = not all(self._kernels(self.ctx.dtype))
 

@@ -75,8 +75,8 @@ def _load_builtins() -> None:
     if not _builtins_loaded:
         _builtins_loaded = True
         from . import (attention, basic, block, conv_attention, delta_rule, diff_attention,  # noqa: F401
-                       filtered_attention, gated_delta, latent_attention, linear_recurrence, moe, normed_attention,
-                       short_conv, side_by_side, stream_join)
+                       filtered_attention, gated_delta, latent_attention, linear_recurrence, matrix_memory, moe,
+                       normed_attention, short_conv, side_by_side, stream_join)
 
 
 def part_class(kind: str, name: str) -> type:

@@ -48,7 +48,9 @@ class ModelSpec:
     `rejoin_runs`: places in `order` before which the embedding's output (the
     stream as it entered the first layer) is added to the stream again. `join` with
     `join_runs`: a part of the "join" registry that makes a new stream of the stream and
-    the embedding's output before those places in `order` (the first place too, if listed)."""
+    the embedding's output before those places in `order` (the first place too, if listed).
+    `max_positions`: the most tokens a sequence can hold, for a model with a table of positions
+    (None: no such bound)."""
 
     hidden_size: int
     vocab_size: int
@@ -59,6 +61,7 @@ class ModelSpec:
     head: PartSpec
     eos_token_ids: tuple[int, ...] = ()
     max_position_embeddings: int | None = None
+    max_positions: int | None = None
     cache_per_run: bool = False
     rejoin_runs: tuple[int, ...] = ()
     join: PartSpec | None = None
@@ -83,7 +86,8 @@ class TensorNeed:
 class KVCacheNeed:
     """A mixer that keeps keys and values: per token `n_kv_heads * head_dim` keys
     and as many values. `window` = None keeps every token; a number keeps only the
-    last `window` tokens readable, and pages wholly before them are given back.
+    last `window` tokens readable, and pages wholly before them are given back;
+    `keep_first` tokens at a sequence's start stay readable besides (their pages stay).
     `n_heads` is the number of query heads that read the cache; the cache manager
     sizes the optional per-page attention-mass accumulators by it. `planes` = 2 keeps
     keys and values; 1 keeps one row per token that serves as both (a mixer that caches
@@ -94,6 +98,7 @@ class KVCacheNeed:
     window: int | None = None
     n_heads: int = 0
     planes: int = 2
+    keep_first: int = 0
 
 
 @dataclasses.dataclass(frozen=True)
