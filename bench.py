@@ -1324,6 +1324,210 @@ def pakarax_kernels(width: int, pk: dict) -> dict:
     return out
 
 
+def zemarax_config(width: int, layers: int, vocab: int = 32000) -> dict:
+    """A Zemarax model at a real model's layer sizes: the layers cycle through latent attention (16 heads over a latent of 128,
+    queries through a latent of width / 4; every second one reads the latents of the first), attention (heads of 64 in groups
+    of four, a window of 1,024 beside four kept tokens) and a matrix memory (heads of 64 x 128, as wide as the model); a dense
+    gated feed-forward of 8/3 x width alternates with 16 routed experts of size width (2 chosen) beside a shared expert of
+    2 x width (the same active size)."""
+    heads, kv = width // 64, max(1, width // 256)
+    mlps = [{"kind": "dense", "ff": (8 * width // 3 + 255) // 256 * 256},
+            {"kind": "moe", "expert": {"ff": width}, "shared": {"ff": 2 * width}, "router": {"experts": 16, "top": 2}}]
+    latent = {"heads": 16, "dim": width // 16, "vdim": width // 16, "q_rank": width // 4, "kv_rank": 128,
+              "scale": (width // 16) ** -0.5}
+    mixers = [("latent_attention", latent),
+              ("attention", {"heads": heads, "kv_heads": kv, "dim": 64, "vdim": 64, "scale": 0.125,
+                             "mask": {"size": 1024, "keep_first": 4}}),
+              ("mlstm", {"heads": width // 128, "dim": 64, "vdim": 128, "gate_cap": 15.0})]
+    out = []
+    for i in range(layers):
+        kind, mixer = mixers[i % 3]
+        if kind == "latent_attention" and i % 6 == 3:
+            mixer = {**mixer, "kv_from": i - 3}
+        out.append({"type": kind, "mixer": mixer, "mlp": mlps[i % 2]})
+    return {"architecture": "Zemarax", "vocab": vocab, "width": width, "max_positions": 8192, "norm": {"eps": 1e-6},
+            "embedding": {"scale": width ** 0.5, "bigram": {"buckets": 65521, "mul_prev": 31, "mul_cur": 7}},
+            "logit_scale": 0.5, "layers": out}
+
+
+def zemarax_kernels(width: int, pk: dict) -> dict:
+    """The Zemarax design's kernels alone at one layer's sizes, each beside the like kernel of the Llama layer (or of the
+    design named): milliseconds, algorithmic bytes or FLOPs, fraction of the copy bandwidth."""
+    import torch
+
+    from pulsarlm_b200.kernels import ops
+
+    dev, bf = "cuda:0", torch.bfloat16
+    out: dict = {}
+
+    def note(name, ms, nbytes=None, flops=None):
+        out[name] = {"ms": ms}
+        if nbytes is not None:
+            out[name].update(bytes=nbytes, frac_of_hbm=nbytes / (ms / 1e3) / 1e9 / pk["hbm_gbs"])
+        if flops is not None:
+            out[name].update(tflops=flops / (ms / 1e3) / 1e12, frac_of_bf16=flops / (ms / 1e3) / 1e12 / pk["bf16_tflops"])
+
+    def f32(*shape):
+        return torch.randn(shape, device=dev)
+
+    def b16(*shape):
+        return f32(*shape).to(bf)
+
+    heads, kv, hd, page = width // 64, max(1, width // 256), 64, 16
+    experts, top, ff = 16, 2, width
+    mh, md, mv = width // 128, 64, 128
+    w1, w2 = f32(width), f32(width)
+    embed, pairs, places = b16(32000, width), b16(65522, width), b16(8192, width)
+    qn, kn = torch.ones(hd, device=dev), torch.ones(hd, device=dev)
+    gates, gate_bias, norm = b16(2 * mh, width), (f32(mh), f32(mh)), torch.ones(mh * mv, device=dev)
+    q_rank, rank = width // 4, 128
+    wq, wc = torch.ones(q_rank, device=dev), torch.ones(rank, device=dev)
+    router, router_shared, bias = f32(experts, width), f32(experts + 1, width), f32(experts)
+    up = b16(experts, ff, width)
+    for tokens, entries in ((2048, 1), (8, 8), (64, 64)):
+        tag = f"T{tokens}_E{entries}"
+        per = tokens // entries
+        entry = torch.arange(entries, dtype=torch.int32, device=dev).repeat_interleave(per)
+        slots = torch.arange(entries, dtype=torch.int32, device=dev)
+        first = torch.arange(0, tokens, per, dtype=torch.int32, device=dev)
+        count = torch.full((entries,), per, dtype=torch.int32, device=dev)
+        pos = torch.arange(8, per + 8, dtype=torch.int32, device=dev).repeat(entries)
+        n_pages = entries * ((per + 8) // page + 1)
+        table = torch.arange(n_pages, dtype=torch.int32, device=dev).view(entries, -1)
+        ids = torch.randint(0, 32000, (tokens,), dtype=torch.int32, device=dev)
+        last = torch.zeros(entries + 1, dtype=torch.int32, device=dev)
+        stream, y = f32(tokens, width), b16(tokens, width)
+        h = torch.empty((tokens, width), dtype=bf, device=dev)
+        note(f"pair_embed_scaled_positions_{tag}",
+             time_kernel(lambda: ops.pair_embed(embed, pairs, ids, pos, entry, slots, last, stream, 31, 7, per == 1, None, 45.0,
+                                                places)), tokens * width * (6 + 4))
+        note(f"embed_{tag} (Llama)", time_kernel(lambda: ops.embed(embed, ids, stream)), tokens * width * (2 + 4))
+        note(f"add_normed_rmsnorm_{tag}", time_kernel(lambda: ops.add_normed_rmsnorm(stream, y, w1, 1.0, 1e-6, w2, 1e-6, h)),
+             tokens * width * (8 + 2 + 2))
+        note(f"add_rmsnorm_{tag} (Llama)", time_kernel(lambda: ops.add_rmsnorm(stream, y, w1, 1e-6, h)),
+             tokens * width * (8 + 2 + 2))
+        # the windowed layer between projection and cache
+        proj = b16(tokens, (heads + 2 * kv) * hd)
+        pools = torch.zeros((2, n_pages, kv, page, hd), dtype=bf, device=dev)
+        q_out = torch.empty((tokens, heads, hd), dtype=bf, device=dev)
+        q, k, v = (proj[:, :heads * hd].view(tokens, heads, hd), proj[:, heads * hd:(heads + kv) * hd].view(tokens, kv, hd),
+                   proj[:, (heads + kv) * hd:].view(tokens, kv, hd))
+        moved = tokens * (heads * hd * 2 * 2 + kv * hd * 2 * 4)
+        note(f"norm_rope_mix_write_per_head_{tag}",
+             time_kernel(lambda: ops.norm_rope_mix_write(q, k, v, None, 0.0, q_out, pos, entry, table, pools[0], pools[1], page,
+                                                         None, 0, "per_head", qn, kn, 1e-6, None, proj.stride(0), None)), moved)
+        inv = torch.rand(hd // 2, dtype=torch.float64, device=dev)
+        note(f"rope_kv_write_{tag} (Llama)",
+             time_kernel(lambda: ops.rope_kv_write(q, k, v, pos, entry, table, pools[0], pools[1], page, inv, hd, None)), moved)
+        # the latents
+        down = b16(tokens, q_rank + rank)
+        pool = torch.zeros((n_pages, 1, page, rank), dtype=bf, device=dev)
+        c_q = torch.empty((tokens, q_rank), dtype=bf, device=dev)
+        note(f"latent_norms_{tag}",
+             time_kernel(lambda: ops.latent_norms(down[:, :q_rank], wq, c_q, down[:, q_rank:], wc, 1e-6, pos, entry, table, pool,
+                                                  page)), tokens * (q_rank + rank) * 4)
+        note(f"norm_write_paged_{tag} (Rerilorn, the cached latent alone)",
+             time_kernel(lambda: ops.norm_write_paged(down[:, q_rank:], wc, 1e-6, pos, entry, table, pool, page)),
+             tokens * rank * 4)
+        # the matrix memory
+        cols = b16(tokens, 2 * mh * md + 2 * mh * mv)
+        parts = (cols[:, :mh * md], cols[:, mh * md:2 * mh * md], cols[:, 2 * mh * md:2 * mh * md + mh * mv],
+                 cols[:, 2 * mh * md + mh * mv:])
+        states = torch.zeros((entries, mh, ops.matrix_memory_head_floats(md, mv)), device=dev)
+        res = torch.empty((tokens, mh * mv), dtype=bf, device=dev)
+        fixed = (gate_bias, 15.0, norm, 1e-6, md ** -0.5, states)
+        traffic = tokens * (cols.shape[1] + mh * mv) * 2 + 2 * states.numel() * 4
+        logits = f32(tokens, 2 * mh)
+        if per > 1:
+            size = ops.matrix_memory_chunk_tokens()
+            chunks = torch.tensor([(r, min(size, tokens - r), 0, int(r + size >= tokens)) for r in range(0, tokens, size)],
+                                  dtype=torch.int32, device=dev)
+            spans = torch.tensor([(0, chunks.shape[0], 0, 0)], dtype=torch.int32, device=dev)
+            note(f"matrix_memory_chunks_{tag}",
+                 time_kernel(lambda: ops.matrix_memory_chunks(parts, cols.stride(0), logits, *fixed, slots, chunks, spans, res, mh,
+                                                              md, mv)), traffic + logits.numel() * 4,
+                 tokens * mh * (2.0 * 64 * md + 2.0 * 64 * mv + 4.0 * md * mv))
+            note(f"matrix_memory_walk_{tag}",
+                 time_kernel(lambda: ops.matrix_memory_walk(parts, cols.stride(0), logits, *fixed, first, count, slots, entry, res,
+                                                            mh, md, mv)), traffic + logits.numel() * 4)
+        else:
+            note(f"matrix_memory_step_{tag}",
+                 time_kernel(lambda: ops.matrix_memory_step(parts, cols.stride(0), y, gates, *fixed, slots, entry, res, mh, md,
+                                                            mv)), traffic + gates.numel() * 2 + tokens * width * 2)
+        nh = width // 64
+        qk = b16(tokens, 3 * nh * 64)
+        delta_states = torch.zeros((entries, nh, 64, 64), device=dev)
+        a_log, dt, dn = f32(nh), f32(nh * 64), torch.ones(64, device=dev)
+        b_pre, a_pre, g_pre = b16(tokens, nh), b16(tokens, nh * 64), b16(tokens, nh * 64)
+        note(f"gated_delta_{tag} (Bunosun)",
+             time_kernel(lambda: ops.gated_delta(qk[:, :nh * 64], qk[:, nh * 64:2 * nh * 64], qk[:, 2 * nh * 64:], b_pre, a_pre,
+                                                 g_pre, a_log, dt, dn, delta_states, first, count, slots, res, nh, nh, 64, 64,
+                                                 1e-6, 0.125, 1e-6)),
+             tokens * width * 12 + 2 * delta_states.numel() * 4)
+        # router, activation, experts pair by pair
+        shared = torch.empty(tokens, device=dev)
+        route_bytes = tokens * width * 2 + experts * width * 4
+        note(f"moe_route_biased_shared_{tag}",
+             time_kernel(lambda: ops.moe_route(h, router_shared, None, top, 1, 1, False, 1, True, shared, bias)), route_bytes)
+        note(f"moe_route_softmax_{tag} (Bunosun)", time_kernel(lambda: ops.moe_route(h, router, None, top, 1, 1)), route_bytes)
+        z = b16(tokens * top, ff)
+        act = torch.empty_like(z)
+        note(f"bias_act_gelu_{tag}", time_kernel(lambda: ops.bias_act(z, None, act, "gelu")), z.numel() * 4)
+        note(f"bias_act_relu2_{tag} (Puvirax)", time_kernel(lambda: ops.bias_act(z, None, act, "relu2")), z.numel() * 4)
+        if tokens <= 8:
+            chosen, _ = ops.moe_route(h, router, None, top, 1, 1)
+            used = int(chosen.unique().numel())
+            for what in ("gelu", "relu2"):
+                note(f"moe_up_{what}_{tag}" + (" (Puvirax)" if what == "relu2" else ""),
+                     time_kernel(lambda: ops.moe_up(h, up, chosen, act, what)), used * ff * width * 2)
+    # attention of 64 single tokens with 2,048 keys: window, kept tokens and sinks beside the Llama layer's windowed
+    # attention; 16 heads over latents of 128 with a sink beside the same with Rerilorn's extras
+    sinks, keys, batch = f32(heads), 2048, 64
+    n_pages = batch * keys // page
+    table = torch.arange(n_pages, dtype=torch.int32, device=dev).view(batch, keys // page)
+    pos = torch.full((batch,), keys - 1, dtype=torch.int32, device=dev)
+    ent = torch.arange(batch, dtype=torch.int32, device=dev)
+    q, kvp = b16(batch, heads, hd), b16(2, n_pages, kv, page, hd)
+    res = torch.empty_like(q)
+    for splits in (1, 4):
+        scratch = torch.empty(ops.attention_decode_scratch_floats(batch, heads, hd, splits), device=dev)
+        for what, ex in (("kept, sink", ops.attention_extras(q, sinks, None, False, keep_first=4)), ("Llama", None)):
+            note(f"attention_decode_b64_w1024_splits{splits} ({what})",
+                 time_kernel(lambda: ops.attention_decode(q, kvp[0], kvp[1], table, pos, ent, res, page, 1024, 0.125, splits,
+                                                          scratch, extras=ex)), batch * 1024 * kv * hd * 4)
+    q, latent, gate, lsinks = b16(batch, 16, rank), b16(n_pages, 1, page, rank), b16(batch, 16), f32(16)
+    res = torch.empty_like(q)
+    for splits in (1, 4):
+        scratch = torch.empty(ops.attention_decode_scratch_floats(batch, 16, rank, splits), device=dev)
+        for what, ex in (("sink", ops.attention_extras(q, lsinks, None, False)),
+                         ("Rerilorn", ops.attention_extras(q, lsinks, gate, True))):
+            note(f"attention_decode_latent_b64_k2048_splits{splits} ({what})",
+                 time_kernel(lambda: ops.attention_decode(q, latent, latent, table, pos, ent, res, page, None, 0.125, splits,
+                                                          scratch, extras=ex)), batch * keys * rank * 2)
+    tokens = 2048
+    n_pages = tokens // page
+    table = torch.arange(n_pages, dtype=torch.int32, device=dev).view(1, n_pages)
+    rows = ops.attention_prefill_tile_rows()
+    tiles = torch.tensor([(r, min(rows, tokens - r), r, 0) for r in range(tokens - rows, -1, -rows)], dtype=torch.int32, device=dev)
+    q, kvp = b16(tokens, heads, hd), b16(n_pages, 2, kv, page, hd)
+    res = torch.empty_like(q)
+    for window in (1024, None):
+        flops = 4.0 * width * sum(min(p + 1, window or tokens) for p in range(tokens))
+        for what, sk, keep in (("kept, sink", sinks, 4), ("Llama", None, 0)):
+            note(f"attention_prefill_tcgen05_T2048_{'w1024' if window else 'causal'} ({what})",
+                 time_kernel(lambda: ops.attention_prefill_tcgen05(q, kvp[:, 0], kvp[:, 1], table, tiles, res, page, window, 0.125,
+                                                                   sinks=sk, keep_first=keep if window else 0)), None, flops)
+    q, latent, gate = b16(tokens, 16, rank), b16(n_pages, 1, page, rank), b16(tokens, 16)
+    res = torch.empty_like(q)
+    flops = 4.0 * 16 * rank * tokens * (tokens + 1) / 2
+    for what, ex in (("sink", ops.attention_extras(q, lsinks, None, False)),
+                     ("Rerilorn", ops.attention_extras(q, lsinks, gate, True)), ("plain", None)):
+        note(f"attention_prefill_latent_T2048 ({what})",
+             time_kernel(lambda: ops.attention_prefill(q, latent, latent, table, tiles, res, page, None, 0.125, extras=ex)), None,
+             flops)
+    return out
+
+
 def run_design(args) -> dict:
     """Prefill and decode throughput of the named design at a few sizes beside the Llama
     decoder at the same width, depth and vocabulary (random weights), and the design's own
@@ -1341,7 +1545,7 @@ def run_design(args) -> dict:
     with ClockSampler() as clocks:
         for width, layers in ((1024, 6), (2048, 6), (4096, 3)):
             mine = {"bunosun": bunosun_config, "rerilorn": rerilorn_config, "simetar": simetar_config,
-                    "puvirax": puvirax_config, "pakarax": pakarax_config}[args.design](width, layers)
+                    "puvirax": puvirax_config, "pakarax": pakarax_config, "zemarax": zemarax_config}[args.design](width, layers)
             for name, cfg in ((args.design, mine), ("llama", llama_config_like(width, layers))):
                 vocab = cfg.get("vocab", cfg.get("vocab_size"))
                 n_pages = (batch * (context + 256) + 4 * prompt) // PAGE_SIZE
@@ -1378,7 +1582,7 @@ def run_design(args) -> dict:
                 gc.collect()
                 torch.cuda.empty_cache()
         kernels = {"bunosun": bunosun_kernels, "rerilorn": design_kernels, "simetar": simetar_kernels,
-                   "puvirax": puvirax_kernels, "pakarax": pakarax_kernels}[args.design](2048, pk)
+                   "puvirax": puvirax_kernels, "pakarax": pakarax_kernels, "zemarax": zemarax_kernels}[args.design](2048, pk)
     summary = clocks.summary()
     return {"metric": f"prefill and decode tok/s of the {args.design.capitalize()} design beside the Llama decoder at "
                       f"equal sizes",
@@ -1392,8 +1596,8 @@ def run_design(args) -> dict:
 
 def main() -> int:
     p = argparse.ArgumentParser()
-    p.add_argument("--design", default="llama", choices=["llama", "rerilorn", "bunosun", "simetar", "puvirax", "pakarax"],
-                   help="llama: the headline workload (the default); rerilorn, bunosun, simetar, puvirax, pakarax: that design's "
+    p.add_argument("--design", default="llama", choices=["llama", "rerilorn", "bunosun", "simetar", "puvirax", "pakarax", "zemarax"],
+                   help="llama: the headline workload (the default); any other name: that design's "
                         "prefill and decode throughput at a few sizes beside the Llama decoder at equal sizes, and its kernels alone")
     p.add_argument("--gpus", type=int, default=1)
     p.add_argument("--steps", type=int, default=128)
@@ -1416,7 +1620,7 @@ def main() -> int:
         print(f"bench.py measures a single-GPU engine: --gpus {args.gpus} is not supported, run with --gpus 1")
         return 2
     args.warmup = max(3, args.warmup)
-    if args.design in ("rerilorn", "bunosun", "simetar", "puvirax", "pakarax"):
+    if args.design != "llama":
         args.steps = min(args.steps, 64)
         print(json.dumps(run_design(args)))
         return 0
