@@ -1520,6 +1520,9 @@ def zemarax_kernels(width: int, pk: dict) -> dict:
     q, latent, gate = b16(tokens, 16, rank), b16(n_pages, 1, page, rank), b16(tokens, 16)
     res = torch.empty_like(q)
     flops = 4.0 * 16 * rank * tokens * (tokens + 1) / 2
+    note("attention_prefill_tcgen05_latent_T2048 (sink)",
+         time_kernel(lambda: ops.attention_prefill_tcgen05(q, latent, latent, table, tiles, res, page, None, 0.125, sinks=lsinks)),
+         None, flops)
     for what, ex in (("sink", ops.attention_extras(q, lsinks, None, False)),
                      ("Rerilorn", ops.attention_extras(q, lsinks, gate, True)), ("plain", None)):
         note(f"attention_prefill_latent_T2048 ({what})",

@@ -35,7 +35,8 @@
 // word, stops, lets loads in flight land, frees its tensor memory and returns.
 //
 // Takes head_dim 64 or 128 and pages that are multiples of 16 tokens in the cache
-// manager's layout [page][K,V][kv head][slot][dim]; other shapes go to the mma.sync
+// manager's layouts [page][K,V][kv head][slot][dim] and [page][kv head][slot][dim] (one row per token that is read
+// as key and as value: a cached latent); other shapes go to the mma.sync
 // kernel in attention_prefill.cu. The reference's counterpart: attn_prefill_tc_kernel,
 // pulsarlm-core/inc/pulsarlm/kernels/paged_prefill.cuh:58-328.
 #include <type_traits>
@@ -60,6 +61,7 @@ struct TcPrefillParams {
     int64_t out_row_stride;
     int group;
     int n_kv_heads;
+    int planes;  // rows a page keeps per token and kv head: 2 (key, value) or 1 (one row that serves as both)
     int page_size;
     int n_pages;
     int window;
@@ -317,7 +319,7 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
                 const int key = __shfl_sync(0xffffffffu, my_key, from);
                 const int page = __shfl_sync(0xffffffffu, my_page, from);
                 if (lane < kPieces * kHalves * 2) {
-                    const int row = ((page * 2) * p.n_kv_heads + kv_head) * p.page_size + key % p.page_size;
+                    const int row = ((page * p.planes) * p.n_kv_heads + kv_head) * p.page_size + key % p.page_size;
                     const int at = h * (kKeys * 128) + piece * (kPiece * 128);
                     tma_load_2d((is_v ? v_s : k_s) + at, is_v ? &map_v : &map_k, h * 64, row, &kv_full[stage]);
                 }
@@ -916,6 +918,14 @@ PL_API int pl_attention_prefill_tcgen05_supports(int head_dim, int page_size, in
         page_stride == 2 * static_cast<int64_t>(n_kv_heads) * head_stride && q_row_stride % 8 == 0;
 }
 
+// 1 when the kernel takes pages that keep one row per token and kv head, read as key and as value (v_pool == k_pool).
+PL_API int pl_attention_prefill_tcgen05_supports_shared(int head_dim, int page_size, int n_kv_heads, int64_t page_stride,
+                                                        int64_t head_stride, int64_t q_row_stride, int dtype) {
+    return dtype == PL_BF16 && (head_dim == 64 || head_dim == 128) && page_size % kPiece == 0 &&
+        head_stride == static_cast<int64_t>(page_size) * head_dim && page_stride == n_kv_heads * head_stride &&
+        q_row_stride % 8 == 0;
+}
+
 // Rows per tile that the kernel can take for this GQA group: with an odd group a CTA
 // works on one head and takes a tile twice as long (its halves share K and V the way
 // two heads of an even group do).
@@ -928,7 +938,8 @@ PL_API int64_t pl_attention_prefill_scratch_floats(int n_tokens, int n_heads, in
 
 // As pl_attention_prefill (tiles of up to 128 rows), on tcgen05. The pools must be
 // the two halves of one [pages][2][kv heads][page][head_dim] tensor: v_pool is
-// k_pool + kv_heads * page * head_dim elements. With n_splits > 1 (at most 32) every
+// k_pool + kv_heads * page * head_dim elements; or one [pages][kv heads][page][head_dim] tensor whose rows serve as
+// keys and as values (v_pool == k_pool; no attention mass). With n_splits > 1 (at most 32) every
 // tile's keys are shared out over that many CTAs and merged by a second kernel
 // through `scratch` (pl_attention_prefill_scratch_floats floats, 16-byte aligned).
 // `wide` (odd groups only; ignored for even ones): the tiles have up to 256 rows
@@ -944,11 +955,12 @@ static int run_tc_prefill(const void* q, int64_t q_row_stride, int n_tokens, con
     PL_REQUIRE(n_tiles >= 0 && n_heads > 0 && n_kv_heads > 0 && n_heads % n_kv_heads == 0 && n_tokens > 0,
                "attention_prefill_tcgen05: bad sizes tiles=%d heads=%d kv_heads=%d tokens=%d", n_tiles, n_heads,
                n_kv_heads, n_tokens);
-    PL_REQUIRE(pl_attention_prefill_tcgen05_supports(head_dim, page_size, n_kv_heads, page_stride, head_stride,
-                                                     q_row_stride, PL_BF16),
+    const bool shared = v_pool == k_pool;
+    PL_REQUIRE((shared ? pl_attention_prefill_tcgen05_supports_shared : pl_attention_prefill_tcgen05_supports)(
+                   head_dim, page_size, n_kv_heads, page_stride, head_stride, q_row_stride, PL_BF16),
                "attention_prefill_tcgen05: unsupported shape or cache layout (head_dim=%d page=%d)", head_dim,
                page_size);
-    PL_REQUIRE(static_cast<const __nv_bfloat16*>(v_pool) ==
+    PL_REQUIRE(shared || static_cast<const __nv_bfloat16*>(v_pool) ==
                    static_cast<const __nv_bfloat16*>(k_pool) + n_kv_heads * head_stride,
                "attention_prefill_tcgen05: v_pool must follow k_pool inside each page");
     PL_REQUIRE((reinterpret_cast<uintptr_t>(q) & 15) == 0 && (reinterpret_cast<uintptr_t>(k_pool) & 15) == 0 &&
@@ -969,11 +981,12 @@ static int run_tc_prefill(const void* q, int64_t q_row_stride, int n_tokens, con
     }
     // Rows of the pool: (page, K or V, kv head, slot); the V map starts one K block in
     // and so has that many rows fewer.
-    const int64_t rows = static_cast<int64_t>(n_pages) * 2 * n_kv_heads * page_size;
+    const int planes = shared ? 1 : 2;
+    const int64_t rows = static_cast<int64_t>(n_pages) * planes * n_kv_heads * page_size;
     if (const int code = make_map(&mk, k_pool, rows, head_dim, head_dim, kPiece, 64)) {
         return code;
     }
-    if (const int code = make_map(&mv, v_pool, rows - static_cast<int64_t>(n_kv_heads) * page_size, head_dim,
+    if (const int code = make_map(&mv, v_pool, rows - static_cast<int64_t>(planes - 1) * n_kv_heads * page_size, head_dim,
                                   head_dim, kPiece, 64)) {
         return code;
     }
@@ -987,6 +1000,7 @@ static int run_tc_prefill(const void* q, int64_t q_row_stride, int n_tokens, con
     p.out_row_stride = out_row_stride;
     p.group = n_heads / n_kv_heads;
     p.n_kv_heads = n_kv_heads;
+    p.planes = planes;
     p.page_size = page_size;
     p.n_pages = n_pages;
     p.window = window;
@@ -1010,6 +1024,7 @@ static int run_tc_prefill(const void* q, int64_t q_row_stride, int n_tokens, con
     p.keep_first = window > 0 && keep_first > 0 ? keep_first : 0;
     PL_REQUIRE((slopes == nullptr && sinks == nullptr && p.keep_first == 0) || (bias == nullptr && mass == nullptr),
                "attention_prefill_tcgen05: a linear bias, sinks and kept first keys are taken without a table and without attention mass");
+    PL_REQUIRE(!shared || mass == nullptr, "attention_prefill_tcgen05: no attention mass over rows that are keys and values");
     PL_REQUIRE(slopes == nullptr || p.keep_first == 0, "attention_prefill_tcgen05: kept first keys are not taken with a linear bias");
     const bool reach = slopes == nullptr && (sinks != nullptr || p.keep_first > 0);
     if (bias != nullptr) {

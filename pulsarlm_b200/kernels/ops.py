@@ -25,7 +25,7 @@ _PTR = ctypes.c_void_p
 _lib = None
 _lock = threading.Lock()
 
-ABI_VERSION = 31
+ABI_VERSION = 32
 
 DTYPE_CODE = {torch.float32: 0, torch.bfloat16: 1}
 
@@ -83,6 +83,7 @@ _SIGNATURES = {
     "pl_attention_prefill_tcgen05_reach": [_PTR, _I64, _I32, _PTR, _PTR, _I64, _I64, _I32, _I32, _PTR, _I32, _PTR, _I32,
                                            _PTR, _I64, _I32, _I32, _I32, _I32, _F32, _I32, _PTR, _PTR, _I32, _PTR, _PTR],
     "pl_attention_prefill_tcgen05_tile_rows": [_I32],
+    "pl_attention_prefill_tcgen05_supports_shared": [_I32, _I32, _I32, _I64, _I64, _I64, _I32],
     "pl_attention_prefill_tcgen05_supports": [_I32, _I32, _I32, _I64, _I64, _I64, _I32],
     "pl_attention_prefill_tile_rows": [],
     "pl_gemm_bf16_pair_supports": [_I32, _I32, _I32, _I64, _I64],
@@ -1584,6 +1585,14 @@ def attention_prefill(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tenso
           ctypes.byref(extras) if extras is not None else None, _p(status), _stream())
 
 
+def attention_prefill_tcgen05_supports_shared(head_dim: int, n_heads: int, k_pool: torch.Tensor, page_size: int) -> bool:
+    """Whether the tcgen05 kernel takes dense queries [T, n_heads, head_dim] over pages whose rows are read as keys and as
+    values (one pool for both)."""
+    return bool(library().pl_attention_prefill_tcgen05_supports_shared(
+        head_dim, page_size, k_pool.shape[1], k_pool.stride(0), k_pool.stride(1), n_heads * head_dim,
+        DTYPE_CODE.get(k_pool.dtype, -1)))
+
+
 def attention_prefill_tcgen05_supports(q: torch.Tensor, k_pool: torch.Tensor, page_size: int) -> bool:
     """Whether the tcgen05 kernel for prompt portions takes this shape and cache layout."""
     return bool(library().pl_attention_prefill_tcgen05_supports(
@@ -1623,7 +1632,8 @@ def attention_prefill_tcgen05(q: torch.Tensor, k_pool: torch.Tensor, v_pool: tor
                               mass: tuple | None = None, distance_bias: torch.Tensor | None = None,
                               distance_slopes: torch.Tensor | None = None, sinks: torch.Tensor | None = None,
                               keep_first: int = 0) -> None:
-    """As attention_prefill, on the tcgen05 tensor cores. `distance_bias` fp32 [nh, rows] (even GQA groups, no
+    """As attention_prefill, on the tcgen05 tensor cores (k_pool and v_pool the halves of the pages, or one pool whose
+    rows are both: see attention_prefill_tcgen05_supports_shared). `distance_bias` fp32 [nh, rows] (even GQA groups, no
     wide tiles, no mass): entry min(distance, rows - 1) of a head's row joins its scaled scores. `distance_slopes` fp32
     [nh] (no mass; an odd group takes narrow and wide tiles alike): slopes[h] * distance is taken off head h's scaled
     scores. `sinks` fp32 [nh] (no mass, no table) join the denominators as exp(sinks[h]); keep_first (with a window;

@@ -8,7 +8,7 @@ import numpy as np
 import torch
 
 from ..kernels import ops
-from .attention import KVBinding, decode_splits
+from .attention import KVBinding, decode_splits, prefill_splits
 from .linear import linear
 from .registry import BuildContext, Part, build_part, register_part
 from .spec import KVCacheNeed, PartSpec, TensorNeed
@@ -93,6 +93,7 @@ class LatentAttention(Part):
         self.up_k = self.up_v = self.o = self.latent_norm = self.sink = None
         self.cache: KVBinding | None = None
         self._tensor_cores: tuple[bool, bool] | None = None
+        self._tcgen05: bool | None = None
 
     @classmethod
     def tensor_needs(cls, spec: PartSpec) -> dict[str, TensorNeed]:
@@ -199,6 +200,16 @@ class LatentAttention(Part):
                 ops.attention_prefill_supports(self.row, self.cache.page_size, dtype))
         return self._tensor_cores
 
+    def _on_tcgen05(self) -> bool:
+        """Whether prompt portions take the tcgen05 kernel: rows of 64 or 128, no gate per head, softmax weights in one
+        bfloat16 term (else the tiled mma.sync kernel)."""
+        if self._tcgen05 is None:
+            self._tcgen05 = (not CUDA_CORES_ONLY and self.ctx.dtype == torch.bfloat16 and not self.split_weights
+                             and self.gate_kind != "head"
+                             and ops.attention_prefill_tcgen05_supports_shared(self.row, self.n_heads, self.cache.k_pool,
+                                                                               self.cache.page_size))
+        return self._tcgen05
+
     def slow_path_note(self) -> str | None:
         if self.cache is None or self.ctx.dtype != torch.bfloat16 or all(self._kernels()):
             return None
@@ -209,19 +220,21 @@ class LatentAttention(Part):
     def plan_key(self):
         if self.cache is None:
             return None
-        return ("latent attention", self.cache.page_size, self.row, self.n_heads, self.window, self.ctx.dtype)
+        return ("latent attention", self.cache.page_size, self.row, self.n_heads, self.window, self.ctx.dtype,
+                self._on_tcgen05())
 
     def plan_step(self, step) -> dict:
         """The tile list of the prompt-portion kernel (int32 [tiles, 4] rows of {first token
         row, rows, position of the first row, block-table row}, the tiles that read the most
         keys first) and the most keys a single token reads."""
         decode_kernel, prefill_kernel = self._kernels()
-        plan: dict = {"tiles": None, "max_context": 0}
+        plan: dict = {"tiles": None, "max_context": 0, "max_keys": 0}
         if decode_kernel and step.n_decode:
             plan["max_context"] = step.context_bound if step.fixed_shape else max(step.context_lens[: step.n_decode])
         if not prefill_kernel or step.n_decode == step.n_entries:
             return plan
-        rows = ops.attention_prefill_tile_rows()
+        rows = (ops.attention_prefill_tcgen05_tile_rows(self.n_heads) if self._on_tcgen05()
+                else ops.attention_prefill_tile_rows())
         tiles = []
         for e in range(step.n_decode, step.n_entries):
             n, at = step.query_lens[e], step.first_rows[e]
@@ -229,13 +242,14 @@ class LatentAttention(Part):
             tiles += [(at + r, min(rows, n - r), start + r, e) for r in range(0, n, rows)]
         tiles.sort(key=lambda t: -(min(t[2] + t[1], self.window + t[1]) if self.window else t[2] + t[1]))
         plan["tiles"] = np.array(tiles, dtype=np.int32).reshape(len(tiles), 4)
+        plan["max_keys"] = max((t[2] + t[1] for t in tiles), default=0)
         return plan
 
     def attend(self, q: torch.Tensor, out: torch.Tensor, table: torch.Tensor, batch, gate) -> None:
         """out[t, h] = gate * sum_j p_j c_j over the latents in reach of token t. In bfloat16 the
         batch's leading single tokens go to the split-key tensor-core kernel and prompt
-        portions to the tiled one, both with the sink and the gate in their last step and the
-        softmax weights kept in two bfloat16 terms; float32, and shapes those kernels do not
+        portions to the tcgen05 one (`_on_tcgen05`) or the tiled one, with the sink and the gate in their
+        last step and the softmax weights kept in one or two bfloat16 terms (`split_weights`); float32, and shapes those kernels do not
         take, attend on the CUDA-core kernel."""
         cache = self.cache
         tokens = q.shape[0]
@@ -261,6 +275,20 @@ class LatentAttention(Part):
         tiles = plan.get("tiles")
         if prefill_kernel and tiles is not None and n_decode == int(batch.n_decode):
             # (the tile list covers exactly the tokens after the leading single tokens)
+            if self._on_tcgen05():
+                odd = self.n_heads % 2 == 1   # (a head per CTA and tiles of up to twice the rows, else two heads)
+                max_keys = int(plan["max_keys"])
+                if self.window:
+                    max_keys = min(max_keys, self.window + ops.attention_prefill_tile_rows())
+                splits = prefill_splits(tiles.shape[0] * (self.n_heads if odd else self.n_heads // 2), max_keys,
+                                        tokens - n_decode, self.n_heads, self.row, q.device)
+                scratch = None
+                if splits > 1:
+                    scratch = torch.empty(ops.attention_prefill_scratch_floats(tokens, self.n_heads, self.row, splits),
+                                          dtype=torch.float32, device=q.device)
+                ops.attention_prefill_tcgen05(q, cache.k_pool, cache.v_pool, table, tiles, out, cache.page_size, self.window,
+                                              self.scale, batch.status, splits, scratch, odd, sinks=self.sink)
+                return
             ops.attention_prefill(q, cache.k_pool, cache.v_pool, table, tiles, out, cache.page_size, self.window,
                                   self.scale, batch.status, extras=ops.attention_extras(q, self.sink, gate, self.split_weights))
             return

@@ -229,6 +229,37 @@ def test_kept_first_keys_and_sinks_on_the_tensor_core_kernels(dim, heads, kv, wi
                     assert plain.relative_error_of(out.cpu(), want) < 1e-2, ("prompt rows on tcgen05", name, rows, splits)
 
 
+@pytest.mark.parametrize("rank,heads", [(64, 4), (128, 16), (64, 3), (128, 5), (64, 1)])
+@pytest.mark.parametrize("spike", [None, 0, 15, 100])
+def test_rows_that_are_keys_and_values_on_tcgen05(rank, heads, spike):
+    """Prompt rows over one pool (a cached latent), a sink per head, one key at a chosen place that stands out."""
+    ops = _ops()
+    page, scale, dtype, lengths = 16, 0.25, torch.bfloat16, [300, 33, 16, 129]
+    spans = [(0, 170, 300), (3, 0, 129), (1, 32, 33), (2, 0, 16)]
+    gen = torch.Generator().manual_seed(rank + heads)
+    queries = [(e, p) for e, lo, hi in spans for p in range(lo, hi)]
+    table, keys, _, q_full, pools = _attention_case(gen, lengths, heads, 1, rank, page, dtype,
+                                                    lambda p: [] if spike is None else [spike], [(0, 299), (3, 128)])
+    sink = torch.randn(heads, generator=gen)
+    want = _wanted(keys, keys, q_full, scale, None, 0, sink, queries)
+    q, pool = torch.stack([q_full[e][p] for e, p in queries]).to(DEV), pools[:, 0].contiguous()
+    assert ops.attention_prefill_tcgen05_supports_shared(rank, heads, pool, page)
+    tiles, at, rows = [], 0, ops.attention_prefill_tcgen05_tile_rows(heads)
+    for e, lo, hi in spans:
+        tiles += [(at + r, min(rows, hi - lo - r), lo + r, e) for r in range(0, hi - lo, rows)]
+        at += hi - lo
+    status = torch.zeros(1, dtype=torch.int32, device=DEV)
+    for with_sink in (True, False):
+        wanted = want if with_sink else _wanted(keys, keys, q_full, scale, None, 0, None, queries)
+        for splits in (1, 3):
+            scratch = torch.empty(ops.attention_prefill_scratch_floats(q.shape[0], heads, rank, splits), dtype=torch.float32,
+                                  device=DEV) if splits > 1 else None
+            out = torch.empty_like(q)
+            ops.attention_prefill_tcgen05(q, pool, pool, table.to(DEV), _i32(tiles), out, page, None, scale, status, splits,
+                                          scratch, heads % 2 == 1, sinks=sink.to(DEV) if with_sink else None)
+            assert int(status.item()) == 0 and plain.relative_error_of(out.cpu(), wanted) < 1e-2, (with_sink, splits)
+
+
 # --------------------------------------------------------------------------- matrix memory
 
 def _memory_case(gen, steps, heads, dim, vdim, hidden, dtype, forget=3.0):
