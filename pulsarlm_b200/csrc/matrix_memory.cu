@@ -379,6 +379,7 @@ __global__ void __launch_bounds__(kChunkThreads) matrix_memory_sums_kernel(const
     if (blockIdx.x == 0) {
         for (int d = threadIdx.x; d < p.dim; d += kChunkThreads) {
             float n = 0.0f;
+#pragma unroll 8
             for (int s = 0; s < rows; ++s) {
                 n = fmaf(w_s[s], __bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(
                                      k_s + swizzled(s, d >> 3, row_bytes) + (d & 7) * 2)), n);
@@ -448,6 +449,7 @@ __global__ void __launch_bounds__(kChainThreads) matrix_memory_chain_kernel(cons
 __global__ void __launch_bounds__(kChunkThreads) matrix_memory_outputs_kernel(const ChunkParams c) {
     extern __shared__ __align__(128) unsigned char smem[];
     __shared__ float b_s[kChunk], a_s[kChunk], m_s[kChunk], qn_s[kChunk];
+    __shared__ __align__(16) float n_s[256];  // n_0
     __shared__ float square_s[8][kChunk];  // [rank][row]
     if (gridDim.x > 1) {
         cluster_arrive_all();  // "this CTA runs": waited for before anything is stored into a peer
@@ -500,6 +502,10 @@ __global__ void __launch_bounds__(kChunkThreads) matrix_memory_outputs_kernel(co
             head_state(p, p.slots[chunk.z], head)[p.dim * p.vdim + p.dim] = total + fmaxf(m0, best);
         }
     }
+    for (int d = threadIdx.x * 4; d < p.dim; d += kChunkThreads * 4) {
+        *reinterpret_cast<float4*>(n_s + d) = *reinterpret_cast<const float4*>(entering + p.dim * p.vdim + d);
+    }
+#pragma unroll 4
     for (int i = threadIdx.x; i < p.dim * 8; i += kChunkThreads) {
         const int d = i >> 3, ch = i & 7;
         float x[8] = {};
@@ -516,14 +522,13 @@ __global__ void __launch_bounds__(kChunkThreads) matrix_memory_outputs_kernel(co
     {
         // q . n_0: two threads a row, each every second 16-byte piece
         const int r = threadIdx.x >> 1, half = threadIdx.x & 1;
-        const float* n0 = entering + p.dim * p.vdim;
         float dot = 0.0f;
         for (int ch = half; ch < p.dim / 8; ch += 2) {
             float x[8];
             unpack8(*reinterpret_cast<const uint4*>(q_s + swizzled(r, ch, row_bytes)), x);
 #pragma unroll
             for (int j = 0; j < 8; ++j) {
-                dot = fmaf(x[j], n0[ch * 8 + j], dot);
+                dot = fmaf(x[j], n_s[ch * 8 + j], dot);
             }
         }
         dot += __shfl_xor_sync(0xffffffffu, dot, 1);
