@@ -166,7 +166,7 @@ def test_kept_first_keys_on_the_cuda_core_kernel(window, keep, dtype):
         assert int(status.item()) == 0 and plain.relative_error_of(out.cpu(), want) < _bar(dtype), name
 
 
-@pytest.mark.parametrize("dim,heads,kv", [(32, 6, 2), (64, 4, 2), (64, 3, 3), (80, 4, 2), (128, 8, 1), (128, 3, 1)])
+@pytest.mark.parametrize("dim,heads,kv", [(32, 6, 2), (64, 8, 4), (64, 3, 3), (80, 6, 3), (128, 8, 1), (128, 3, 1)])
 @pytest.mark.parametrize("window,keep", REACH)
 def test_kept_first_keys_and_sinks_on_the_tensor_core_kernels(dim, heads, kv, window, keep):
     """bfloat16 single tokens (any number of key shares) and prompt rows (mma.sync, and tcgen05 where it takes the
@@ -316,7 +316,7 @@ def _memory_steps(part, sequences, schedule, slot_of):
     return {r: torch.cat(x) for r, x in got.items()}
 
 
-SHAPES = [(4, 32, 64), (3, 16, 24), (2, 64, 128), (5, 6, 10), (2, 48, 80), (1, 128, 64), (2, 256, 40), (3, 8, 4), (2, 20, 200),
+SHAPES = [(6, 32, 64), (3, 16, 24), (2, 64, 128), (5, 6, 10), (2, 48, 80), (1, 128, 64), (2, 256, 40), (3, 8, 4), (2, 20, 200),
           (1, 96, 512), (2, 40, 1)]
 
 
